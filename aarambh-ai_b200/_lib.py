@@ -14,7 +14,7 @@ LIB_PATH = os.path.join(HERE, "libaarambh_b200.so")
 OK = 0
 F32, F16, BF16 = 0, 1, 2
 KV_F32, KV_BF16, KV_INT8 = 0, 1, 2
-FMT_I8, FMT_I4_AFFINE, FMT_Q4KM, FMT_W4A16 = 0, 1, 2, 3
+FMT_I8, FMT_I4_AFFINE, FMT_Q4KM, FMT_W4A16, FMT_BF16 = 0, 1, 2, 3, 4
 
 STATUS_NAMES = {
     0: "OK", -1: "BAD_SHAPE", -2: "BAD_ALIGN", -3: "BAD_DTYPE", -4: "CAPACITY", -5: "CUDA_ERROR",
@@ -47,6 +47,7 @@ SIGNATURES = {
     "ab2_version": ([], _i),
     "ab2_last_error": ([], C.c_char_p),
     "ab2_device_status": ([C.POINTER(_i)], _i),
+    "ab2_qweight_from_bf16": ([_pp, _p, _i, _i], _i),
     "ab2_qweight_from_i8_tensor": ([_pp, _p, _f, _i, _i], _i),
     "ab2_qweight_from_i8_channel": ([_pp, _p, _p, _i, _i], _i),
     "ab2_qweight_from_i4_affine": ([_pp, _p, _p, _p, _i, _i, _i], _i),
@@ -71,6 +72,9 @@ SIGNATURES = {
     "ab2_argmax": ([_p, _i, _i, _i, _p, _p], _i),
     "ab2_embedding_forward": ([_p, _p, _i, _p, _i, _p], _i),
     "ab2_kv_create": ([_pp, _i, _i, _i, _i, _i, _i, _i], _i),
+    "ab2_kv_create_stack": ([_pp, _p, _i, _i, _i, _i, _i], _i),
+    "ab2_kv_save_row": ([_p, _i, _p], _i),
+    "ab2_kv_has_state": ([_p, C.POINTER(_i)], _i),
     "ab2_kv_destroy": ([_p], _i),
     "ab2_kv_update": ([_p, _p, _p, _i, _i, _i, _i, _p], _i),
     "ab2_kv_append": ([_p, _i, _p, _p, _i, _i, _i, _i, _p, _p, _p, _i, _p], _i),
@@ -86,6 +90,7 @@ SIGNATURES = {
     "ab2_attention_cached": ([_p, _i, _p, _p, _i, _i, _i, _f, _i, _p], _i),
     "ab2_attention_causal": ([_p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _p], _i),
     "ab2_model_create": ([_pp, _p, _i, _i], _i),
+    "ab2_model_create_stack": ([_pp, _p, _p, _i, _i], _i),
     "ab2_model_destroy": ([_p], _i),
     "ab2_model_set_linear": ([_p, _i, _i, _p], _i),
     "ab2_model_set_norm": ([_p, _i, _i, _p], _i),
@@ -118,6 +123,18 @@ class ModelConfig(C.Structure):
     _fields_ = [("n_layers", _i), ("d_model", _i), ("n_heads", _i), ("n_kv_heads", _i),
                 ("head_dim", _i), ("ffn_hidden", _i), ("vocab", _i), ("max_seq", _i),
                 ("rms_eps", _f), ("rope_theta", C.c_double), ("tied", _i)]
+
+
+MIX_ATTENTION, MIX_LIGHTNING = 0, 1
+FFN_NONE, FFN_MOE = 0, 1
+
+
+class LayerSpec(C.Structure):
+    """ab2_layer_spec."""
+    _fields_ = [("mixer", _i), ("heads", _i), ("dim", _i), ("vdim", _i), ("kv_heads", _i), ("window", _i),
+                ("rot_dims", _i), ("rot_base", C.c_double), ("qk_norm", _i), ("scale", _f), ("v_mix", _i),
+                ("v_lambda", _f), ("decay", C.POINTER(_f)), ("ffn", _i), ("experts", _i), ("top", _i), ("ff", _i),
+                ("limit", _f)]
 
 
 def _declare():

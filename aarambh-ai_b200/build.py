@@ -68,5 +68,14 @@ def build(force: bool = False, verbose: bool = False) -> str:
     return LIB
 
 
+def build_locked() -> str:
+    """``build`` under a file lock, for programs that may start together in a fresh checkout."""
+    import fcntl
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build()
+
+
 if __name__ == "__main__":
     print(build(force="--force" in sys.argv, verbose="--verbose" in sys.argv))

@@ -376,6 +376,7 @@ __global__ void attn_rowwise_kernel(const T *__restrict__ q, const T *__restrict
 static int check_attention(const ab2_kv *kv, int layer, const void *q, const void *out, int S, int row0,
                            int nrows, ab2_dtype dtype) {
     AB2_REQUIRE(kv && q && out, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(!kv->layers, AB2_ERR_UNSUPPORTED, "the cache of a layer stack is read by its model's steps");
     AB2_REQUIRE(layer >= 0 && layer < kv->L, AB2_ERR_BAD_SHAPE, "layer %d outside the cache's %d layers", layer, kv->L);
     AB2_REQUIRE(S > 0 && nrows > 0 && row0 >= 0 && row0 + nrows <= kv->B, AB2_ERR_BAD_SHAPE,
                 "rows %d..%d outside the cache batch %d", row0, row0 + nrows, kv->B);

@@ -45,7 +45,8 @@ enum Format : int {
     FMT_I8 = 0,         // int8 codes [N][K], f32 scale per row
     FMT_I4_AFFINE = 1,  // nibbles [N*K/2], f32 scale + f32 zero per flat group
     FMT_Q4KM = 2,       // nibbles [ceil(N*K/256)*128], (f16 scale, f16 min) per 256-block
-    FMT_W4A16 = 3       // tile-major blocks of code and parameter words (w4a16_layout.cuh)
+    FMT_W4A16 = 3,      // tile-major blocks of code and parameter words (w4a16_layout.cuh)
+    FMT_BF16 = 4        // dense bf16 [N][K], no parameters
 };
 
 }  // namespace ab2

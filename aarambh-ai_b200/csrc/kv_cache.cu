@@ -7,6 +7,7 @@
 // reference keeps [batch, capacity, kv_heads, head_dim]
 // (crates/aarambh-studio-nn/src/kvcache.rs:349-368) and transposes on every
 // step (crates/aarambh-studio-nn/src/attention.rs:272-276).
+#include <algorithm>
 #include <cfloat>
 #include <cstring>
 
@@ -182,7 +183,7 @@ int kv_append_device(ab2_kv *kv, int layer, const void *k, const void *v, long l
 int kv_commit_device(ab2_kv *kv, int S, int row0, int nrows, cudaStream_t s) {
     kv_advance_kernel<<<(nrows + 127) / 128, 128, 0, s>>>(kv->lens_dev, kv->rows_on ? kv->rows_dev : nullptr, row0, nrows, S);
     AB2_LAUNCH_CHECK();
-    for (int i = 0; i < nrows; ++i) kv->lens_host[kv_row_host(kv, row0, i)] += S;
+    for (int i = 0; i < nrows; ++i) kv_advance_host(kv, kv_row_host(kv, row0, i), S);
     return AB2_OK;
 }
 
@@ -234,8 +235,101 @@ AB2_API int ab2_kv_create(ab2_kv **out, int n_layers, int batch, int capacity, i
     return AB2_OK;
 }
 
+// Bytes of one sequence's share of a stack layer.
+static size_t layer_row_bytes(const KvLayer &l, bool value, int esz) {
+    return (size_t)l.kvh * l.cap * (value ? l.vds : l.kds) * esz;
+}
+static size_t layer_state_elems(const KvLayer &l) { return (size_t)l.kvh * l.kd * l.vd; }
+
+AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n_layers, int batch, int capacity,
+                                int max_step, ab2_kv_dtype dtype) {
+    AB2_REQUIRE(out != nullptr && specs != nullptr, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(n_layers > 0 && batch > 0 && capacity > 0 && max_step > 0, AB2_ERR_BAD_SHAPE, "KV cache dimensions must be positive");
+    AB2_REQUIRE(dtype == AB2_KV_F32 || dtype == AB2_KV_BF16, AB2_ERR_BAD_DTYPE, "a layer stack caches f32 or bf16, got %d", (int)dtype);
+    ab2_kv *kv = new ab2_kv();
+    memset(kv, 0, sizeof(*kv));
+    kv->L = n_layers; kv->B = batch; kv->cap = capacity; kv->dtype = dtype;
+    kv->layers = new KvLayer[n_layers]();
+    kv->high_host = new int[batch]();
+    kv->saved_len = new int[batch];
+    for (int i = 0; i < batch; ++i) kv->saved_len[i] = -1;
+    const int esz = (int)kv_elem_size(dtype);
+    kv->max_splits = AB2_KV_MAX_SPLITS;
+    size_t part = 0, heads = 0;
+    cudaError_t e = cudaSuccess;
+    for (int i = 0; i < n_layers && e == cudaSuccess; ++i) {
+        const ab2_layer_spec &sp = specs[i];
+        KvLayer &l = kv->layers[i];
+        l.recurrent = sp.mixer == AB2_MIX_LIGHTNING;
+        l.kd = sp.dim; l.vd = sp.vdim;
+        if (l.recurrent) {
+            l.kvh = sp.heads;
+            e = cudaMalloc((void **)&l.state, (size_t)batch * layer_state_elems(l) * 4);
+            if (e == cudaSuccess) e = cudaMemset(l.state, 0, (size_t)batch * layer_state_elems(l) * 4);
+            continue;
+        }
+        l.kvh = sp.kv_heads;
+        l.kds = (l.kd + 7) / 8 * 8; l.vds = (l.vd + 7) / 8 * 8;
+        // a step of max_step tokens is appended before its queries look back a whole window
+        l.window = sp.window > 0 ? std::min(sp.window, capacity) : capacity;
+        l.cap = (int)std::min<long long>(capacity, (long long)l.window - 1 + max_step);
+        for (int which = 0; which < 2 && e == cudaSuccess; ++which) {
+            void **p = which ? &l.v : &l.k;
+            e = cudaMalloc(p, (size_t)batch * layer_row_bytes(l, which, esz));
+            if (e == cudaSuccess) e = cudaMemset(*p, 0, (size_t)batch * layer_row_bytes(l, which, esz));
+        }
+        part = std::max(part, (size_t)sp.heads * l.vd);
+        heads = std::max(heads, (size_t)sp.heads);
+    }
+    if (e == cudaSuccess) e = cudaMalloc((void **)&kv->lens_dev, (size_t)batch * 4);
+    if (e == cudaSuccess) e = cudaMemset(kv->lens_dev, 0, (size_t)batch * 4);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->lens_host, (size_t)batch * 4);
+    if (e == cudaSuccess) e = cudaMalloc((void **)&kv->rows_dev, (size_t)batch * 4);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->rows_host, (size_t)batch * 4);
+    kv->part_acc_bytes = (size_t)batch * kv->max_splits * part * 4;
+    kv->part_ml_bytes = (size_t)batch * kv->max_splits * heads * 2 * 4;
+    if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_acc, kv->part_acc_bytes);
+    if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_ml, kv->part_ml_bytes);
+    if (e != cudaSuccess) {
+        ab2_kv_destroy(kv);
+        return fail(AB2_ERR_CUDA, "KV cache allocation failed: %s", cudaGetErrorString(e));
+    }
+    memset(kv->lens_host, 0, (size_t)batch * 4);
+    *out = kv;
+    return AB2_OK;
+}
+
+// Remembers the recurrent states of `row` at its current length (the keys and values need no copy:
+// their slots stay intact, see ab2_kv_truncate).
+AB2_API int ab2_kv_save_row(ab2_kv *kv, int row, ab2_stream stream) {
+    AB2_REQUIRE(kv != nullptr, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(row >= 0 && row < kv->B, AB2_ERR_BAD_SHAPE, "row %d outside the cache batch %d", row, kv->B);
+    if (!kv->layers) return AB2_OK;
+    for (int i = 0; i < kv->L; ++i) {
+        KvLayer &l = kv->layers[i];
+        if (!l.recurrent) continue;
+        const size_t n = layer_state_elems(l);
+        if (!l.saved) AB2_CUDA(cudaMalloc((void **)&l.saved, (size_t)kv->B * n * 4));
+        AB2_CUDA(cudaMemcpyAsync(l.saved + row * n, l.state + row * n, n * 4, cudaMemcpyDeviceToDevice, (cudaStream_t)stream));
+    }
+    kv->saved_len[row] = kv->lens_host[row];
+    return AB2_OK;
+}
+
+AB2_API int ab2_kv_has_state(const ab2_kv *kv, int *has_state) {
+    AB2_REQUIRE(kv != nullptr && has_state != nullptr, AB2_ERR_BAD_ARG, "null argument");
+    *has_state = 0;
+    for (int i = 0; kv->layers && i < kv->L; ++i) *has_state |= kv->layers[i].recurrent;
+    return AB2_OK;
+}
+
 AB2_API int ab2_kv_destroy(ab2_kv *kv) {
     if (!kv) return AB2_OK;
+    for (int i = 0; kv->layers && i < kv->L; ++i) {
+        cudaFree(kv->layers[i].k); cudaFree(kv->layers[i].v);
+        cudaFree(kv->layers[i].state); cudaFree(kv->layers[i].saved);
+    }
+    delete[] kv->layers; delete[] kv->high_host; delete[] kv->saved_len;
     cudaFree(kv->k); cudaFree(kv->v); cudaFree(kv->ks); cudaFree(kv->vs); cudaFree(kv->lens_dev);
     cudaFree(kv->part_acc); cudaFree(kv->part_ml); cudaFree(kv->counters);
     if (kv->lens_host) cudaFreeHost(kv->lens_host);
@@ -248,6 +342,7 @@ AB2_API int ab2_kv_destroy(ab2_kv *kv) {
 static int check_append(const ab2_kv *kv, int layer, const void *k, const void *v, int S, int row0,
                         int nrows, ab2_dtype dtype) {
     AB2_REQUIRE(kv && k && v, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(!kv->layers, AB2_ERR_UNSUPPORTED, "the cache of a layer stack is filled by its model's steps");
     AB2_REQUIRE(layer >= 0 && layer < kv->L, AB2_ERR_BAD_SHAPE, "layer %d outside the cache's %d layers", layer, kv->L);
     AB2_REQUIRE(S > 0 && nrows > 0 && row0 >= 0 && row0 + nrows <= kv->B, AB2_ERR_BAD_SHAPE,
                 "rows %d..%d outside the cache batch %d", row0, row0 + nrows, kv->B);
@@ -298,6 +393,26 @@ AB2_API int ab2_kv_truncate(ab2_kv *kv, int row, int new_len, ab2_stream stream)
     AB2_REQUIRE(row >= 0 && row < kv->B, AB2_ERR_BAD_SHAPE, "row %d outside the cache batch %d", row, kv->B);
     AB2_REQUIRE(new_len >= 0 && new_len <= kv->lens_host[row], AB2_ERR_CAPACITY,
                 "cannot grow KV cache from %d to %d with truncate", kv->lens_host[row], new_len);
+    if (kv->layers && new_len != 0 && new_len != kv->lens_host[row]) {
+        // Every layer must still hold what a sequence of new_len tokens would: a ring that has not
+        // written over the window before new_len, a recurrent state saved at that length.
+        for (int i = 0; i < kv->L; ++i) {
+            KvLayer &l = kv->layers[i];
+            if (l.recurrent)
+                AB2_REQUIRE(kv->saved_len[row] == new_len, AB2_ERR_UNSUPPORTED,
+                            "row %d has a recurrent state: it can be cut to 0 or to the length of ab2_kv_save_row, not to %d", row, new_len);
+            else
+                AB2_REQUIRE(kv->high_host[row] - l.cap <= std::max(0, new_len - l.window + 1), AB2_ERR_CAPACITY,
+                            "row %d held %d tokens: its ring of %d no longer has the window before %d", row, kv->high_host[row], l.cap, new_len);
+        }
+        for (int i = 0; i < kv->L; ++i) {
+            KvLayer &l = kv->layers[i];
+            if (!l.recurrent) continue;
+            const size_t n = layer_state_elems(l);
+            AB2_CUDA(cudaMemcpyAsync(l.state + row * n, l.saved + row * n, n * 4, cudaMemcpyDeviceToDevice, (cudaStream_t)stream));
+        }
+    }
+    if (kv->layers && new_len == 0) { kv->high_host[row] = 0; kv->saved_len[row] = -1; }
     kv->lens_host[row] = new_len;
     AB2_CUDA(cudaMemcpyAsync(kv->lens_dev + row, kv->lens_host + row, 4, cudaMemcpyHostToDevice, (cudaStream_t)stream));
     AB2_CUDA(cudaStreamSynchronize((cudaStream_t)stream));
@@ -307,6 +422,8 @@ AB2_API int ab2_kv_truncate(ab2_kv *kv, int row, int new_len, ab2_stream stream)
 AB2_API int ab2_kv_clear(ab2_kv *kv, ab2_stream stream) {
     AB2_REQUIRE(kv != nullptr, AB2_ERR_BAD_ARG, "null argument");
     memset(kv->lens_host, 0, (size_t)kv->B * 4);
+    if (kv->layers)
+        for (int r = 0; r < kv->B; ++r) { kv->high_host[r] = 0; kv->saved_len[r] = -1; }
     AB2_CUDA(cudaMemsetAsync(kv->lens_dev, 0, (size_t)kv->B * 4, (cudaStream_t)stream));
     return AB2_OK;
 }
@@ -324,8 +441,53 @@ AB2_API int ab2_kv_capacity(const ab2_kv *kv, int *capacity) {
     return AB2_OK;
 }
 
+static int clone_stack(ab2_kv **out, const ab2_kv *src, cudaStream_t s) {
+    ab2_kv *kv = new ab2_kv();
+    *kv = *src;
+    kv->layers = new KvLayer[src->L]();
+    kv->high_host = new int[src->B]();
+    kv->saved_len = new int[src->B];
+    for (int i = 0; i < src->B; ++i) { kv->high_host[i] = src->high_host[i]; kv->saved_len[i] = -1; }
+    kv->lens_dev = kv->lens_host = kv->rows_dev = kv->rows_host = nullptr;
+    kv->part_acc = kv->part_ml = nullptr;
+    kv->rows_on = false;
+    cudaError_t e = cudaSuccess;
+    auto dup = [&](void **dst, const void *from, size_t bytes, bool contents) {
+        if (e == cudaSuccess && from) e = cudaMalloc(dst, bytes);
+        if (e == cudaSuccess && from && contents) e = cudaMemcpyAsync(*dst, from, bytes, cudaMemcpyDeviceToDevice, s);
+    };
+    const int esz = (int)kv_elem_size(src->dtype);
+    for (int i = 0; i < src->L; ++i) {
+        const KvLayer &a = src->layers[i];
+        KvLayer &b = kv->layers[i];
+        b = a;
+        b.k = b.v = nullptr; b.state = b.saved = nullptr;
+        if (a.recurrent) {
+            dup((void **)&b.state, a.state, (size_t)src->B * layer_state_elems(a) * 4, true);
+        } else {
+            dup(&b.k, a.k, (size_t)src->B * layer_row_bytes(a, false, esz), true);
+            dup(&b.v, a.v, (size_t)src->B * layer_row_bytes(a, true, esz), true);
+        }
+    }
+    dup((void **)&kv->lens_dev, src->lens_dev, (size_t)src->B * 4, true);
+    dup((void **)&kv->rows_dev, src->rows_dev, (size_t)src->B * 4, false);
+    dup((void **)&kv->part_acc, src->part_acc, src->part_acc_bytes, false);
+    dup((void **)&kv->part_ml, src->part_ml, src->part_ml_bytes, false);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->lens_host, (size_t)src->B * 4);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->rows_host, (size_t)src->B * 4);
+    if (e == cudaSuccess) e = cudaStreamSynchronize(s);
+    if (e != cudaSuccess) {
+        ab2_kv_destroy(kv);
+        return fail(AB2_ERR_CUDA, "KV cache clone failed: %s", cudaGetErrorString(e));
+    }
+    memcpy(kv->lens_host, src->lens_host, (size_t)src->B * 4);
+    *out = kv;
+    return AB2_OK;
+}
+
 AB2_API int ab2_kv_clone(ab2_kv **out, const ab2_kv *src, ab2_stream stream) {
     AB2_REQUIRE(out != nullptr && src != nullptr, AB2_ERR_BAD_ARG, "null argument");
+    if (src->layers) return clone_stack(out, src, (cudaStream_t)stream);
     int rc = ab2_kv_create(out, src->L, src->B, src->cap, src->kvh, src->hd, src->h, (ab2_kv_dtype)src->dtype);
     if (rc != AB2_OK) return rc;
     ab2_kv *dst = *out;
@@ -352,6 +514,7 @@ AB2_API int ab2_kv_clone(ab2_kv **out, const ab2_kv *src, ab2_stream stream) {
 AB2_API int ab2_kv_read(const ab2_kv *kv, int layer, int row, float *k_out_dev, float *v_out_dev,
                         ab2_stream stream) {
     AB2_REQUIRE(kv && k_out_dev && v_out_dev, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(!kv->layers, AB2_ERR_UNSUPPORTED, "the layers of a stack differ in what they keep: there is no common read-back");
     AB2_REQUIRE(layer >= 0 && layer < kv->L, AB2_ERR_BAD_SHAPE, "layer %d outside the cache's %d layers", layer, kv->L);
     AB2_REQUIRE(row >= 0 && row < kv->B, AB2_ERR_BAD_SHAPE, "row %d outside the cache batch %d", row, kv->B);
     int len = kv->lens_host[row];

@@ -5,6 +5,19 @@
 
 #define AB2_KV_MAX_SPLITS 64
 
+// What one layer of a layer stack keeps per sequence: either the last `cap` keys and values
+// (position p in slot p % cap), or a recurrent state.
+struct KvLayer {
+    bool recurrent;
+    int kvh, kd, vd;      // attention: heads, key and value size; recurrent: heads and the two state dimensions
+    int kds, vds;         // row strides of k and v in elements (multiples of 8; the padding stays zero)
+    int cap;              // ring slots per (sequence, head)
+    int window;           // keys a query may see
+    void *k, *v;          // [B][kvh][cap][kds], [B][kvh][cap][vds]
+    float *state;         // [B][kvh][kd][vd]
+    float *saved;         // same shape: the state ab2_kv_save_row keeps
+};
+
 struct ab2_kv {
     int L, B, cap, kvh, hd, h;
     int dtype;        // ab2_kv_dtype
@@ -22,6 +35,11 @@ struct ab2_kv {
     int *rows_dev;    // [B]
     int *rows_host;   // [B], pinned
     bool rows_on;
+    // Layer stacks: per-layer geometry (null for the uniform cache above, whose k / v are then unused)
+    KvLayer *layers;
+    int *high_host;   // [B] most tokens a row has held since it was last empty (which ring slots are intact)
+    int *saved_len;   // [B] length ab2_kv_save_row recorded, -1 none
+    size_t part_acc_bytes, part_ml_bytes;
 };
 
 namespace ab2 {
@@ -42,7 +60,30 @@ static inline int kv_row_host(const ab2_kv *kv, int row0, int i) {
     return kv->rows_on ? kv->rows_host[row0 + i] : row0 + i;
 }
 
+// The host mirror of a row's length moves on by S tokens.
+static inline void kv_advance_host(ab2_kv *kv, int row, int S) {
+    kv->lens_host[row] += S;
+    if (kv->high_host && kv->high_host[row] < kv->lens_host[row]) kv->high_host[row] = kv->lens_host[row];
+}
+
 KvView kv_view(const ab2_kv *kv, int layer);
+
+// One layer of a stack as kernels receive it.
+struct KvLayerView {
+    KvLayer l;
+    const int *lens;
+    const int *rows;
+};
+__device__ __forceinline__ int kv_row(const KvLayerView &kv, int row0, int i) {
+    return kv.rows ? kv.rows[row0 + i] : row0 + i;
+}
+static inline KvLayerView kv_layer_view(const ab2_kv *kv, int layer) {
+    KvLayerView v;
+    v.l = kv->layers[layer];
+    v.lens = kv->lens_dev;
+    v.rows = kv->rows_on ? kv->rows_dev : nullptr;
+    return v;
+}
 
 // Writes S tokens per row at the rows' current lengths (no advance).  k / v
 // element (row, s, head, d) sits at (row * S + s) * in_stride + head * hd + d.

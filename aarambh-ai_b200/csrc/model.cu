@@ -14,6 +14,7 @@
 #include "common.cuh"
 #include "kv_cache.cuh"
 #include "ops.cuh"
+#include "stack.cuh"
 #include "tp.cuh"
 #include "decode_step_persistent.cuh"
 
@@ -46,6 +47,7 @@ struct StepGraph {
 };
 
 struct ab2_model {
+    ab2::Stack *stack;     // a decoder made of layer specs (stack.cu); null for the dense decoder below
     ab2_model_config cfg;
     ab2_dtype dtype;
     int max_tokens;
@@ -158,6 +160,7 @@ static int norm_linear(ab2_model *m, const ab2_qweight *w, const void *x, const 
 static int forward_launches(ab2_model *m, ab2_kv *kv, const uint32_t *ids, int S, int row0, int nrows,
                             const int *rope_base, int logits_mode, void *logits, uint32_t *argmax_out,
                             int len_hint, cudaStream_t s) {
+    if (m->stack) return stack_forward(m->stack, kv, ids, S, row0, nrows, logits_mode, (float *)logits, argmax_out, len_hint, s);
     const ab2_model_config &c = m->cfg;
     const int T = nrows * S, d = c.d_model, hd = c.head_dim;
     const size_t esz = dtype_size(m->dtype);
@@ -340,8 +343,13 @@ static int check_forward(ab2_model *m, ab2_kv *kv, const void *ids, int S, int r
     AB2_REQUIRE(m->finalized, AB2_ERR_BAD_ARG, "model is not finalised");
     const ab2_model_config &c = m->cfg;
     AB2_REQUIRE(kv->L == c.n_layers, AB2_ERR_BAD_SHAPE, "expected %d cache layers, got %d", c.n_layers, kv->L);
-    AB2_REQUIRE(kv->kvh == c.n_kv_heads && kv->hd == c.head_dim && kv->h == c.n_heads, AB2_ERR_BAD_SHAPE,
-                "KV cache head layout does not match the model");
+    if (m->stack) {
+        int rc = stack_check_cache(m->stack, kv, S);
+        if (rc != AB2_OK) return rc;
+    } else {
+        AB2_REQUIRE(!kv->layers && kv->kvh == c.n_kv_heads && kv->hd == c.head_dim && kv->h == c.n_heads, AB2_ERR_BAD_SHAPE,
+                    "KV cache head layout does not match the model");
+    }
     AB2_REQUIRE(S > 0 && nrows > 0 && row0 >= 0 && row0 + nrows <= kv->B, AB2_ERR_BAD_SHAPE,
                 "rows %d..%d outside the cache batch %d", row0, row0 + nrows, kv->B);
     for (int r = 0; r < nrows; ++r) {
@@ -390,8 +398,21 @@ AB2_API int ab2_model_create(ab2_model **out, const ab2_model_config *cfg, ab2_d
     return AB2_OK;
 }
 
+AB2_API int ab2_model_create_stack(ab2_model **out, const ab2_model_config *cfg, const ab2_layer_spec *specs, ab2_dtype dtype,
+                                   int max_tokens) {
+    AB2_REQUIRE(out && cfg && specs, AB2_ERR_BAD_ARG, "null argument");
+    Stack *st = nullptr;
+    int rc = stack_create(&st, *cfg, specs, dtype, max_tokens);
+    if (rc != AB2_OK) return rc;
+    ab2_model *m = new ab2_model();
+    m->stack = st; m->cfg = *cfg; m->dtype = dtype; m->max_tokens = max_tokens;
+    *out = m;
+    return AB2_OK;
+}
+
 AB2_API int ab2_model_destroy(ab2_model *m) {
     if (!m) return AB2_OK;
+    stack_destroy(m->stack);
     for (auto &g : m->graphs) cudaGraphExecDestroy(g.second.exec);
     persistent_step_destroy(m->persistent);
     for (auto &L : m->layers) {
@@ -409,6 +430,10 @@ AB2_API int ab2_model_destroy(ab2_model *m) {
 
 AB2_API int ab2_model_set_linear(ab2_model *m, int layer, int which, const ab2_qweight *w) {
     AB2_REQUIRE(m && w, AB2_ERR_BAD_ARG, "null argument");
+    if (m->stack) {
+        m->finalized = false;
+        return stack_set_linear(m->stack, layer, which, w);
+    }
     const ab2_model_config &c = m->cfg;
     int N = 0, K = 0;
     if (layer < 0) {
@@ -431,6 +456,7 @@ AB2_API int ab2_model_set_linear(ab2_model *m, int layer, int which, const ab2_q
 
 AB2_API int ab2_model_set_norm(ab2_model *m, int layer, int which, const float *weight) {
     AB2_REQUIRE(m && weight, AB2_ERR_BAD_ARG, "null argument");
+    if (m->stack) return stack_set_norm(m->stack, layer, which, weight);
     const int d = m->cfg.d_model;
     float **slot;
     if (layer < 0) slot = &m->final_norm;
@@ -446,6 +472,14 @@ AB2_API int ab2_model_set_norm(ab2_model *m, int layer, int which, const float *
 AB2_API int ab2_model_finalize(ab2_model *m) {
     AB2_REQUIRE(m != nullptr, AB2_ERR_BAD_ARG, "null argument");
     const ab2_model_config &c = m->cfg;
+    if (m->stack) {
+        int rc = stack_finalize(m->stack);
+        if (rc != AB2_OK) return rc;
+        for (auto &g : m->graphs) cudaGraphExecDestroy(g.second.exec);
+        m->graphs.clear();
+        m->finalized = true;
+        return AB2_OK;
+    }
     AB2_REQUIRE(m->embedding && m->final_norm, AB2_ERR_BAD_ARG, "embedding or final norm not set");
     if (!m->lm_head) {
         AB2_REQUIRE(c.tied, AB2_ERR_BAD_ARG, "lm_head not set and embeddings are not tied");
@@ -542,6 +576,7 @@ AB2_API int ab2_model_finalize(ab2_model *m) {
 
 AB2_API int ab2_model_set_tp(ab2_model *m, ab2_tp *tp) {
     AB2_REQUIRE(m != nullptr, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(!(m->stack && tp), AB2_ERR_UNSUPPORTED, "a layer stack runs on one GPU");
     AB2_REQUIRE(m->x == nullptr, AB2_ERR_BAD_ARG, "set the tensor-parallel context before the model is finalised");
     if (tp) AB2_REQUIRE(m->cfg.vocab % tp->world == 0, AB2_ERR_BAD_SHAPE, "vocab %d is not divisible by the world size %d", m->cfg.vocab, tp->world);
     m->tp = tp;
@@ -550,6 +585,7 @@ AB2_API int ab2_model_set_tp(ab2_model *m, ab2_tp *tp) {
 
 AB2_API int ab2_model_rope_tables(const ab2_model *m, const float **cos_dev, const float **sin_dev) {
     AB2_REQUIRE(m && m->finalized, AB2_ERR_BAD_ARG, "model is not finalised");
+    AB2_REQUIRE(!m->stack, AB2_ERR_UNSUPPORTED, "the layers of a stack have rotations of their own");
     if (cos_dev) *cos_dev = m->cos_t;
     if (sin_dev) *sin_dev = m->sin_t;
     return AB2_OK;
@@ -566,6 +602,7 @@ AB2_API int ab2_model_forward(ab2_model *m, ab2_kv *kv, const uint32_t *ids_dev,
         bool same = true;
         for (int r = 0; r < nrows; ++r) same = same && offsets_host[r] == kv->lens_host[kv_row_host(kv, row0, r)];
         if (!same) {
+            AB2_REQUIRE(!m->stack, AB2_ERR_UNSUPPORTED, "a layer stack takes the cache lengths as offsets");
             AB2_REQUIRE(!kv->rows_on, AB2_ERR_UNSUPPORTED, "a forward over selected rows takes the cache lengths as offsets");
             // explicit seqlen offsets that differ from the cache lengths
             AB2_CUDA(cudaStreamSynchronize(s));
@@ -655,16 +692,19 @@ AB2_API int ab2_model_decode_step(ab2_model *m, ab2_kv *kv, const uint32_t *ids_
     auto it = m->graphs.find(key);
     if (it == m->graphs.end()) {
         cudaGraph_t graph = nullptr;
-        rc = w4a16_prepare_stream(s);  // scratch of the GEMV is allocated outside the capture
+        if (!m->stack) rc = w4a16_prepare_stream(s);  // scratch of the GEMV is allocated outside the capture
         if (rc != AB2_OK) return rc;
         AB2_CUDA(cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal));
-        g_pdl_launch = m->fused_epilogues;  // every kernel of the fast path takes part in the chain
+        g_pdl_launch = m->fused_epilogues || m->stack;  // every kernel of the fast path takes part in the chain
         rc = forward_launches(m, kv, ids_dev, 1, row0, nrows, kv->lens_dev, logits_dev ? 1 : 0, logits_dev, argmax_dev, len_bound, s);
         if (rc == AB2_OK) {
             // lengths advance inside the graph; the host mirror is advanced per replay
             std::vector<int> keep(kv->lens_host, kv->lens_host + kv->B);
+            std::vector<int> high;
+            if (kv->high_host) high.assign(kv->high_host, kv->high_host + kv->B);
             rc = kv_commit_device(kv, 1, row0, nrows, s);
             memcpy(kv->lens_host, keep.data(), (size_t)kv->B * 4);
+            if (kv->high_host) memcpy(kv->high_host, high.data(), (size_t)kv->B * 4);
         }
         g_pdl_launch = false;
         cudaError_t e = cudaStreamEndCapture(s, &graph);
@@ -677,7 +717,7 @@ AB2_API int ab2_model_decode_step(ab2_model *m, ab2_kv *kv, const uint32_t *ids_
         it = m->graphs.emplace(key, sg).first;
     }
     AB2_CUDA(cudaGraphLaunch(it->second.exec, s));
-    for (int i = 0; i < nrows; ++i) kv->lens_host[kv_row_host(kv, row0, i)] += 1;
+    for (int i = 0; i < nrows; ++i) kv_advance_host(kv, kv_row_host(kv, row0, i), 1);
     return AB2_OK;
 }
 

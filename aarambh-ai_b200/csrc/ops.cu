@@ -6,6 +6,7 @@
 
 #include "common.cuh"
 #include "ops.cuh"
+#include "stack.cuh"
 #include "w4a16_layout.cuh"
 
 using namespace ab2;
@@ -149,6 +150,101 @@ int launch_add_rms_norm(void *x, const void *p, const float *w, void *out, int r
     int rc = launch_add(x, p, x, (size_t)rows * d, dtype, s);
     if (rc != AB2_OK) return rc;
     return launch_rms_norm(x, w, out, rows, d, eps, dtype, s);
+}
+
+// ---- normalisation around an f32 residual stream ------------------------------
+// One CTA per token; the row is formed once in shared memory (see ResidualNorm in stack.cuh).
+template <typename T, int MODE>
+__global__ void residual_norm_kernel(ResidualNormArgs a) {
+    extern __shared__ float vrow[];
+    __shared__ float warp_sums[32];
+    const size_t t = blockIdx.x;
+    pdl_wait();
+    pdl_launch_dependents();
+    const float *parts = a.parts + t * (size_t)(MODE == RN_ADD ? a.nparts : 1) * a.d;
+    const float *xsrc = a.x + (MODE == RN_FINAL ? t * a.step + a.step - 1 : t) * (size_t)a.d;
+    uint32_t id = 0;
+    if (MODE == RN_EMBED) {
+        id = a.ids[t];
+        if (id >= (uint32_t)a.vocab) id = a.vocab - 1;  // ids are validated on the host; keep reads in range
+    }
+    float sum = 0.f;
+    const bool vec = (a.d & 3) == 0;
+    if (vec) {
+        for (int i = threadIdx.x; i < a.d / 4; i += blockDim.x) {
+            float4 v;
+            if (MODE == RN_EMBED) {
+                const uint2 e = reinterpret_cast<const uint2 *>(a.table + (size_t)id * a.d)[i];
+                v = make_float4(__uint_as_float(e.x << 16), __uint_as_float(e.x & 0xffff0000u), __uint_as_float(e.y << 16),
+                                __uint_as_float(e.y & 0xffff0000u));
+            } else if (MODE == RN_FINAL) {
+                v = reinterpret_cast<const float4 *>(xsrc)[i];
+            } else {
+                v = reinterpret_cast<const float4 *>(parts)[i];
+                if (MODE == RN_ADD)
+                    for (int p = 1; p < a.nparts; ++p) {
+                        const float4 q = reinterpret_cast<const float4 *>(parts + (size_t)p * a.d)[i];
+                        v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+                    }
+            }
+            reinterpret_cast<float4 *>(vrow)[i] = v;
+            sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
+        }
+    } else {
+        for (int i = threadIdx.x; i < a.d; i += blockDim.x) {
+            float v;
+            if (MODE == RN_EMBED) v = __bfloat162float(a.table[(size_t)id * a.d + i]);
+            else if (MODE == RN_FINAL) v = xsrc[i];
+            else {
+                v = parts[i];
+                if (MODE == RN_ADD)
+                    for (int p = 1; p < a.nparts; ++p) v += parts[(size_t)p * a.d + i];
+            }
+            vrow[i] = v;
+            sum = fmaf(v, v, sum);
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if ((threadIdx.x & 31) == 0) warp_sums[threadIdx.x >> 5] = sum;
+    __syncthreads();
+    sum = 0.f;
+    for (int w = 0; w < (int)(blockDim.x >> 5); ++w) sum += warp_sums[w];
+    const float inv = 1.f / sqrtf(sum / (float)a.d + a.eps);
+    T *out = (T *)a.out + t * (size_t)a.d;
+    const T *gate = (const T *)a.gate + t * (size_t)a.gate_stride;
+    float *x = a.x + t * (size_t)a.d;
+    // a thread reads back the elements it wrote, so the row needs no second barrier
+    const int step = vec ? 4 : 1;
+    for (int i0 = threadIdx.x * step; i0 < a.d; i0 += blockDim.x * step) {
+        for (int j = 0; j < step; ++j) {
+            const int i = i0 + j;
+            float v = vrow[i] * inv * a.w[i];
+            if (MODE == RN_ADD) v += x[i];
+            if (MODE == RN_GATED) v *= to_f32(gate[i]);
+            if (MODE == RN_EMBED || MODE == RN_ADD) x[i] = v;
+            if (a.out != nullptr) out[i] = from_f32<T>(v);
+        }
+    }
+}
+
+template <typename T>
+static cudaError_t launch_residual(const ResidualNormArgs &a, int mode, int rows, cudaStream_t s) {
+    const int threads = std::min(1024, std::max(128, (a.d / 8 + 31) / 32 * 32));
+    const size_t smem = (size_t)a.d * 4;
+    switch (mode) {
+    case RN_EMBED: return launch_kernel(residual_norm_kernel<T, RN_EMBED>, dim3(rows), dim3(threads), smem, s, a);
+    case RN_ADD: return launch_kernel(residual_norm_kernel<T, RN_ADD>, dim3(rows), dim3(threads), smem, s, a);
+    case RN_FINAL: return launch_kernel(residual_norm_kernel<T, RN_FINAL>, dim3(rows), dim3(threads), smem, s, a);
+    default: return launch_kernel(residual_norm_kernel<T, RN_GATED>, dim3(rows), dim3(threads), smem, s, a);
+    }
+}
+
+int launch_residual_norm(const ResidualNormArgs &a, int mode, int rows, ab2_dtype dtype, cudaStream_t s) {
+    AB2_REQUIRE(a.d <= 12000, AB2_ERR_UNSUPPORTED, "rows of %d values exceed the shared memory of the normalisation", a.d);
+    cudaError_t e = dtype == AB2_F32 ? launch_residual<float>(a, mode, rows, s) : launch_residual<__nv_bfloat16>(a, mode, rows, s);
+    if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "normalisation launch failed: %s", cudaGetErrorString(e));
+    return AB2_OK;
 }
 
 // ---- RoPE ------------------------------------------------------------------
@@ -323,7 +419,9 @@ __global__ void embedding_kernel(const uint32_t *__restrict__ ids, int vocab, in
     for (int k = blockIdx.y * blockDim.x + threadIdx.x; k < K; k += gridDim.y * blockDim.x) {
         size_t idx = (size_t)id * K + k;
         float v;
-        if (fmt == FMT_I8) {
+        if (fmt == FMT_BF16) {
+            v = __bfloat162float(((const __nv_bfloat16 *)codes)[idx]);
+        } else if (fmt == FMT_I8) {
             v = __fmul_rn((float)((const int8_t *)codes)[idx], scales[id]);
         } else if (fmt == FMT_I4_AFFINE) {
             uint8_t byte = ((const uint8_t *)codes)[idx >> 1];

@@ -11,6 +11,7 @@
 #include "gemv_w4a16_warp.cuh"
 #include "gemv_w4a16_m1.cuh"
 #include "gemv_w4a16_strip.cuh"
+#include "linear_bf16.cuh"
 
 using namespace ab2;
 
@@ -54,7 +55,8 @@ int qlinear_validate(const ab2_qweight *w, const void *x, int M, ab2_dtype dtype
     AB2_REQUIRE(M > 0, AB2_ERR_BAD_SHAPE, "token count must be positive, got %d", M);
     AB2_REQUIRE(dtype == AB2_F32 || dtype == AB2_F16 || dtype == AB2_BF16, AB2_ERR_BAD_DTYPE,
                 "unsupported activation dtype %d", (int)dtype);
-    AB2_REQUIRE(w->K % 8 == 0, AB2_ERR_BAD_SHAPE, "in_features=%d must be a multiple of 8", w->K);
+    if (w->fmt != FMT_BF16)
+        AB2_REQUIRE(w->K % 8 == 0, AB2_ERR_BAD_SHAPE, "in_features=%d must be a multiple of 8", w->K);
     AB2_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)y & (dtype_size(dtype) - 1)) == 0,
                 AB2_ERR_BAD_ALIGN, "activations must be 16-byte aligned");
     if (w->fmt == FMT_I4_AFFINE)
@@ -409,6 +411,7 @@ bool qlinear_i8_tc_eligible(const ab2_qweight *w, ab2_dtype dtype, int M);
 int qlinear_i8_tc(const ab2_qweight *w, const void *x, int M, void *y, cudaStream_t s);
 
 int qlinear_dispatch(const ab2_qweight *w, const void *x, int M, ab2_dtype dtype, void *y, cudaStream_t s) {
+    if (w->fmt == FMT_BF16) return linear_bf16(w, x, M, dtype, y, LIN_STORE, 0, s);
     if (qlinear_w4a16_mma_eligible(w, dtype)) {
         // Up to 64 tokens: the HBM-bound decode kernels (one token, 2..8 tokens, chunks of 9..32
         // tokens).  The tcgen05 GEMM tiles 128 output channels per CTA, which leaves most SMs

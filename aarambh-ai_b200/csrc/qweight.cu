@@ -120,6 +120,21 @@ static int upload_i8(ab2_qweight **out, const int8_t *codes, const float *scales
     return AB2_OK;
 }
 
+AB2_API int ab2_qweight_from_bf16(ab2_qweight **out, const uint16_t *weight, int N, int K) {
+    AB2_REQUIRE(weight != nullptr, AB2_ERR_BAD_ARG, "weight pointer is null");
+    TRY(alloc_handle(out, FMT_BF16, N, K, K));
+    ab2_qweight *w = *out;
+    w->codes_bytes = (size_t)N * K * 2;
+    TRY_OR_FREE(w, dev_alloc(&w->codes, (w->codes_bytes + 15) / 16 * 16));
+    cudaError_t e = cudaMemcpy(w->codes, weight, w->codes_bytes, cudaMemcpyDefault);
+    if (e != cudaSuccess) {
+        ab2_qweight_destroy(w);
+        *out = nullptr;
+        return fail(AB2_ERR_CUDA, "bf16 weight upload failed: %s", cudaGetErrorString(e));
+    }
+    return AB2_OK;
+}
+
 AB2_API int ab2_qweight_from_i8_tensor(ab2_qweight **out, const int8_t *codes, float scale, int N,
                                        int K) {
     AB2_REQUIRE(codes != nullptr, AB2_ERR_BAD_ARG, "codes pointer is null");
@@ -325,6 +340,9 @@ AB2_API int ab2_qweight_export(const ab2_qweight *w, void *codes, void *scales, 
     AB2_REQUIRE(w != nullptr, AB2_ERR_BAD_ARG, "weight handle is null");
     size_t n = (size_t)w->N * w->K;
     switch (w->fmt) {
+    case FMT_BF16:
+        if (codes) AB2_CUDA(cudaMemcpy(codes, w->codes, w->codes_bytes, cudaMemcpyDefault));
+        break;
     case FMT_I8:
         if (codes) AB2_CUDA(cudaMemcpy(codes, w->codes, n, cudaMemcpyDefault));
         if (scales) AB2_CUDA(cudaMemcpy(scales, w->scales, w->per_tensor ? 4 : (size_t)w->N * 4, cudaMemcpyDefault));
@@ -396,6 +414,7 @@ static QView view_of(const ab2_qweight *w) {
 // no fused multiply-add, same operand order.
 __device__ __forceinline__ float dequant_element(const QView &v, size_t idx) {
     switch (v.fmt) {
+    case FMT_BF16: return __bfloat162float(((const __nv_bfloat16 *)v.codes)[idx]);
     case FMT_I8: {  // dequant.rs:8-16: code as f32 * scale
         float c = (float)((const int8_t *)v.codes)[idx];
         return __fmul_rn(c, v.scales[idx / v.K]);

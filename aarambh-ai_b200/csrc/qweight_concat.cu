@@ -45,6 +45,11 @@ AB2_API int ab2_qweight_concat_rows(ab2_qweight **out, const ab2_qweight *const 
         }
     };
     switch (first->fmt) {
+    case FMT_BF16:
+        w->codes_bytes = (size_t)N * K * 2;
+        copy_parts(&w->codes, w->codes_bytes, [&](const ab2_qweight *p) { return (size_t)p->N * K * 2; },
+                   [](const ab2_qweight *p) { return (const void *)p->codes; });
+        break;
     case FMT_I8:
         w->codes_bytes = (size_t)N * K; w->param_bytes = (size_t)N * 4;
         copy_parts(&w->codes, w->codes_bytes, [&](const ab2_qweight *p) { return (size_t)p->N * K; },

@@ -1,0 +1,89 @@
+// Layer stacks: the parts shared by the mechanisms and the model (internal header).
+#pragma once
+
+#include <vector>
+
+#include "common.cuh"
+#include "kv_cache.cuh"
+#include "linear_bf16.cuh"
+
+namespace ab2 {
+
+// ---- sliding-window attention (attention_window.cu) -----------------------------
+struct WindowPrepArgs {
+    KvLayerView kv;
+    void *qkv;             // [nrows * S][stride]: H query heads, G key heads, G value heads; queries are rewritten
+    long long stride;
+    int S, row0, H, G, dim, vdim, rot_dims, qk_norm;
+    const float *cos_t, *sin_t;  // [positions][rot_dims / 2]
+    float eps;
+    void *v_first;         // [nrows * S][G * vdim]
+    int v_mode;            // 0 values as they are, 1 also keep them in v_first, 2 mix them with v_first
+    float lambda;
+};
+struct WindowAttnArgs {
+    KvLayerView kv;
+    const void *q;         // head h of token t at t * q_stride + h * dim
+    long long q_stride;
+    void *out;             // [nrows * S][H * vdim]
+    int S, row0, H, rep, dim, vdim, nsplit;
+    float scale;
+    float *part_acc, *part_ml;
+};
+// Rotation, normalisation and value mixing of S new tokens per row, which are then stored in the cache.
+int window_prep(const WindowPrepArgs &a, int nrows, ab2_dtype dtype, cudaStream_t s);
+// Attention of the S tokens just stored; max_len bounds the rows' lengths with them.
+int window_attention(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, ab2_dtype dtype, cudaStream_t s);
+
+// ---- lightning attention (linear_attention.cu) ------------------------------------
+struct LightningArgs {
+    KvLayerView kv;
+    const void *qkv;       // [nrows * S][stride]: q, k (heads x dim), v (heads x vdim), activated
+    long long stride;
+    float *out;            // [nrows * S][heads * vdim]
+    int S, row0, H, dim, vdim;
+    const float *decay_pow;  // [heads][LIGHTNING_CHUNK + 1]: powers 0, 1, ... of the head's decay
+};
+constexpr int LIGHTNING_CHUNK = 64;
+int lightning_attention(const LightningArgs &a, int nrows, ab2_dtype dtype, cudaStream_t s);
+
+// ---- normalisation around the f32 residual stream (ops.cu) -------------------------
+// Every form computes RMSNorm(v; w) of one row v per token.
+enum ResidualNorm : int {
+    RN_EMBED = 0,  // v = table[ids[t]];            x = norm
+    RN_ADD = 1,    // v = sum of the token's parts; x += norm
+    RN_FINAL = 2,  // v = x[t * step + step - 1];   out = norm
+    RN_GATED = 3   // v = parts[t];                 out = norm * gate[t]
+};
+struct ResidualNormArgs {
+    const float *w;
+    float eps;
+    int d;
+    const __nv_bfloat16 *table;
+    const uint32_t *ids;
+    int vocab;
+    const float *parts;    // RN_ADD: [T][nparts][d], RN_GATED: [T][d]
+    int nparts, step;
+    const void *gate;      // activation type, row stride gate_stride
+    long long gate_stride;
+    float *x;              // [T][d]
+    void *out;             // activation type; RN_EMBED / RN_ADD: the new x rounded to it (null: not wanted)
+};
+int launch_residual_norm(const ResidualNormArgs &a, int mode, int rows, ab2_dtype dtype, cudaStream_t s);
+
+// ---- mixture of experts (moe.cu) ---------------------------------------------------
+// Scores, choice and sorting of T tokens from router logits [T][E].
+int moe_route(const float *logits, int T, const MoeRoute &r, cudaStream_t s);
+
+// ---- the stack ---------------------------------------------------------------------
+struct Stack;
+int stack_create(Stack **out, const ab2_model_config &cfg, const ab2_layer_spec *specs, ab2_dtype dtype, int max_tokens);
+void stack_destroy(Stack *st);
+int stack_set_linear(Stack *st, int layer, int which, const ab2_qweight *w);
+int stack_set_norm(Stack *st, int layer, int which, const float *weight);
+int stack_finalize(Stack *st);
+int stack_check_cache(const Stack *st, const ab2_kv *kv, int S);
+int stack_forward(Stack *st, ab2_kv *kv, const uint32_t *ids, int S, int row0, int nrows, int logits_mode, float *logits,
+                  uint32_t *argmax_out, int len_hint, cudaStream_t s);
+
+}  // namespace ab2

@@ -35,6 +35,14 @@ class KVCache:
     def with_capacity(cls, capacity, kv_heads, head_dim, n_heads, **kw):
         return cls(capacity, kv_heads, head_dim, n_heads, **kw)
 
+    @classmethod
+    def for_stack(cls, cfg, capacity: int, batch: int, max_step: int, dtype: str):
+        """The cache of a layer stack (``StackConfig``): windows in rings, recurrent states beside them."""
+        specs, _keep = cfg.c_specs()
+        h = C.c_void_p()
+        check(lib.ab2_kv_create_stack(C.byref(h), specs, len(cfg.layers), batch, capacity, max_step, _KV_DTYPES[dtype]))
+        return cls(capacity, 0, 0, 0, batch, len(cfg.layers), dtype, _handle=h.value)
+
     def update(self, k: torch.Tensor, v: torch.Tensor, row0: int = 0):
         """Appends k, v [rows, S, kv_heads, head_dim] and returns the cached tensors
         of the first row touched, dequantised ([len, kv_heads, head_dim])."""
@@ -65,6 +73,16 @@ class KVCache:
 
     def truncate(self, new_len: int, row: int = 0):
         check(lib.ab2_kv_truncate(self._h, row, new_len, stream_ptr()))
+
+    def save_row(self, row: int = 0):
+        """Remembers a row's recurrent states, so that ``truncate`` to its present length can restore them."""
+        check(lib.ab2_kv_save_row(self._h, row, stream_ptr()))
+
+    def has_state(self) -> bool:
+        """Whether a layer keeps a recurrent state (its rows are cut to 0 or to a saved length only)."""
+        n = C.c_int()
+        check(lib.ab2_kv_has_state(self._h, C.byref(n)))
+        return bool(n.value)
 
     def clear(self):
         check(lib.ab2_kv_clear(self._h, stream_ptr()))

@@ -44,42 +44,21 @@ class ModelConfig:
         return cls(32, 4096, 32, 8, 128, 14336, 32000, 1024, tie_embeddings=False)
 
 
-class AarambhModel:
-    """weights: name -> QuantLinear for ``embedding``, optional ``lm_head`` and
-    ``layers.{i}.{wq,wk,wv,wo,w_gate,w_up,w_down}``; name -> f32 tensor for
-    ``final_norm`` and ``layers.{i}.{norm1,norm2}``."""
+class DecoderModel:
+    """The step functions of a decoder handle (``ab2_model``), whatever layers it is made of.
+    A subclass creates the handle and says what cache it takes."""
 
-    def __init__(self, cfg: ModelConfig, weights: dict, dtype: torch.dtype = torch.float32,
-                 max_tokens: int = 512, tp=None):
-        """With ``tp`` (a ``parallel.TensorParallel``), ``cfg`` and ``weights`` are
-        this rank's shard (``parallel.shard_config`` / ``shard_weight``)."""
-        self.cfg, self.dtype, self.weights, self.tp = cfg, dtype, weights, tp
-        c = _CConfig(cfg.n_layers, cfg.d_model, cfg.n_heads, cfg.n_kv_heads, cfg.head_dim, cfg.ffn_hidden,
-                     cfg.vocab_size, cfg.max_seq_len, cfg.rms_norm_eps, cfg.rope_theta,
-                     1 if cfg.tie_embeddings else 0)
+    dtype: torch.dtype            # activation type
+    logits_dtype: torch.dtype     # element type of the logits
+
+    def _create(self, fn, *args):
         h = C.c_void_p()
-        check(lib.ab2_model_create(C.byref(h), C.byref(c), dtype_code(dtype), max_tokens))
+        check(fn(C.byref(h), *args))
         self._h = h
-        if tp is not None:
-            check(lib.ab2_model_set_tp(self._h, tp._h))
-        check(lib.ab2_model_set_linear(self._h, -1, 0, weights["embedding"]._h))
-        if "lm_head" in weights:
-            check(lib.ab2_model_set_linear(self._h, -1, 1, weights["lm_head"]._h))
-        self._norm(-1, 0, weights["final_norm"])
-        for l in range(cfg.n_layers):
-            for which, name in enumerate(LAYER_LINEARS):
-                check(lib.ab2_model_set_linear(self._h, l, which, weights[f"layers.{l}.{name}"]._h))
-            self._norm(l, 0, weights[f"layers.{l}.norm1"])
-            self._norm(l, 1, weights[f"layers.{l}.norm2"])
-        check(lib.ab2_model_finalize(self._h))
 
     def _norm(self, layer, which, w):
         w = w.detach().to(torch.float32).contiguous()
         check(lib.ab2_model_set_norm(self._h, layer, which, w.data_ptr()))
-
-    def empty_kv_cache_with_capacity(self, capacity: int, batch: int = 1, dtype: str = "f32") -> KVCache:
-        c = self.cfg
-        return KVCache(capacity, c.n_kv_heads, c.head_dim, c.n_heads, batch, c.n_layers, dtype)
 
     def _ids(self, token_ids):
         ids = token_ids if isinstance(token_ids, torch.Tensor) else torch.tensor(token_ids)
@@ -96,11 +75,17 @@ class AarambhModel:
         if ids.shape[0] != 1:
             raise _lib.Ab2Error(-1, "forward_with_cache takes one sequence")
         S = ids.shape[1]
-        out = torch.empty((1, 1 if last_only else S, self.cfg.vocab_size), dtype=self.dtype, device="cuda")
+        out = torch.empty((1, 1 if last_only else S, self.cfg.vocab_size), dtype=self.logits_dtype, device="cuda")
         offs = (C.c_int * 1)(seqlen_offset)
         check(lib.ab2_model_forward(self._h, cache._h, ids.data_ptr(), S, row, 1, offs, 1 if last_only else 2,
                                     out.data_ptr(), None, stream_ptr()))
         return out
+
+    def extend_cache(self, token_ids, cache: KVCache, row: int = 0) -> None:
+        """Runs ids [1, S] from the row's cache length on for what they leave in the cache (no logits)."""
+        ids = self._ids(token_ids)
+        check(lib.ab2_model_forward(self._h, cache._h, ids.data_ptr(), ids.shape[1], row, 1, None, 0, None, None,
+                                    stream_ptr()))
 
     def forward_decode_batch(self, token_ids, seqlen_offsets, cache: KVCache, row0: int = 0) -> torch.Tensor:
         """ids [B, 1], offsets [B] -> logits [B, 1, vocab]."""
@@ -110,7 +95,7 @@ class AarambhModel:
         B = ids.shape[0]
         if len(seqlen_offsets) != B:
             raise _lib.Ab2Error(-1, f"batched decode received batch {B} and {len(seqlen_offsets)} offsets")
-        out = torch.empty((B, 1, self.cfg.vocab_size), dtype=self.dtype, device="cuda")
+        out = torch.empty((B, 1, self.cfg.vocab_size), dtype=self.logits_dtype, device="cuda")
         offs = (C.c_int * B)(*[int(o) for o in seqlen_offsets])
         check(lib.ab2_model_forward(self._h, cache._h, ids.data_ptr(), 1, row0, B, offs, 1, out.data_ptr(), None,
                                     stream_ptr()))
@@ -124,7 +109,7 @@ class AarambhModel:
         if ids.shape[1] != 1 or ids.shape[0] != len(rows):
             raise _lib.Ab2Error(-1, f"expected ids [{len(rows)}, 1], got {list(ids.shape)}")
         n = len(rows)
-        out = torch.empty((n, 1, self.cfg.vocab_size), dtype=self.dtype, device="cuda")
+        out = torch.empty((n, 1, self.cfg.vocab_size), dtype=self.logits_dtype, device="cuda")
         check(lib.ab2_model_forward_rows(self._h, cache._h, ids.data_ptr(), 1, (C.c_int * n)(*rows), n, 1,
                                          out.data_ptr(), None, stream_ptr()))
         return out
@@ -173,6 +158,149 @@ class AarambhModel:
         except Exception:
             pass
 
+class AarambhModel(DecoderModel):
+    """weights: name -> QuantLinear for ``embedding``, optional ``lm_head`` and
+    ``layers.{i}.{wq,wk,wv,wo,w_gate,w_up,w_down}``; name -> f32 tensor for
+    ``final_norm`` and ``layers.{i}.{norm1,norm2}``."""
+
+    def __init__(self, cfg: ModelConfig, weights: dict, dtype: torch.dtype = torch.float32,
+                 max_tokens: int = 512, tp=None):
+        """With ``tp`` (a ``parallel.TensorParallel``), ``cfg`` and ``weights`` are
+        this rank's shard (``parallel.shard_config`` / ``shard_weight``)."""
+        self.cfg, self.dtype, self.weights, self.tp = cfg, dtype, weights, tp
+        c = _CConfig(cfg.n_layers, cfg.d_model, cfg.n_heads, cfg.n_kv_heads, cfg.head_dim, cfg.ffn_hidden,
+                     cfg.vocab_size, cfg.max_seq_len, cfg.rms_norm_eps, cfg.rope_theta,
+                     1 if cfg.tie_embeddings else 0)
+        self.max_tokens, self.logits_dtype = max_tokens, dtype
+        self._create(lib.ab2_model_create, C.byref(c), dtype_code(dtype), max_tokens)
+        if tp is not None:
+            check(lib.ab2_model_set_tp(self._h, tp._h))
+        check(lib.ab2_model_set_linear(self._h, -1, 0, weights["embedding"]._h))
+        if "lm_head" in weights:
+            check(lib.ab2_model_set_linear(self._h, -1, 1, weights["lm_head"]._h))
+        self._norm(-1, 0, weights["final_norm"])
+        for l in range(cfg.n_layers):
+            for which, name in enumerate(LAYER_LINEARS):
+                check(lib.ab2_model_set_linear(self._h, l, which, weights[f"layers.{l}.{name}"]._h))
+            self._norm(l, 0, weights[f"layers.{l}.norm1"])
+            self._norm(l, 1, weights[f"layers.{l}.norm2"])
+        check(lib.ab2_model_finalize(self._h))
+
+    kv_dtype = "f32"   # of a cache that names none
+
+    def empty_kv_cache_with_capacity(self, capacity: int, batch: int = 1, dtype: str = "f32") -> KVCache:
+        c = self.cfg
+        return KVCache(capacity, c.n_kv_heads, c.head_dim, c.n_heads, batch, c.n_layers, dtype)
+
+
+@dataclass
+class AttentionMixer:
+    """Grouped-query softmax attention over a sliding window (``window`` keys, 0: all of them)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+    rot_dims: int = 0             # leading dimensions rotated, in adjacent pairs
+    rot_base: float = 10000.0
+    qk_norm: bool = False         # q and k divided by their root mean square after the rotation
+    v_mix: bool = False           # values mixed with those of the stack's first such layer
+    v_lambda: float = 0.0
+
+
+@dataclass
+class LightningMixer:
+    """Linear attention with one decay per head."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+
+
+@dataclass
+class MoeFfn:
+    """Mixture of experts: sigmoid scores that multiply the chosen experts' inputs, clamped gated unit."""
+    experts: int
+    top: int
+    ff: int
+    limit: float
+
+
+@dataclass
+class StackConfig:
+    """A decoder listed layer by layer: ``layers`` holds (mixer, feed-forward or None) pairs."""
+    d_model: int
+    vocab_size: int
+    layers: list
+    max_seq_len: int
+    rms_norm_eps: float = 1e-5
+    tie_embeddings: bool = True
+
+    def c_specs(self):
+        """The layers as an array of ab2_layer_spec (and what it points to)."""
+        arr = (_lib.LayerSpec * len(self.layers))()
+        keep = []
+        for s, (mix, ffn) in zip(arr, self.layers):
+            s.heads, s.dim, s.vdim = mix.heads, mix.dim, mix.vdim
+            if isinstance(mix, LightningMixer):
+                if len(mix.decay) != mix.heads:
+                    raise _lib.Ab2Error(-1, f"{len(mix.decay)} decays for {mix.heads} heads")
+                s.mixer = _lib.MIX_LIGHTNING
+                keep.append((C.c_float * mix.heads)(*mix.decay))
+                s.decay = C.cast(keep[-1], C.POINTER(C.c_float))
+            else:
+                s.mixer = _lib.MIX_ATTENTION
+                s.kv_heads, s.window, s.scale = mix.kv_heads, mix.window, mix.scale
+                s.rot_dims, s.rot_base, s.qk_norm = mix.rot_dims, mix.rot_base, int(mix.qk_norm)
+                s.v_mix, s.v_lambda = int(mix.v_mix), mix.v_lambda
+            if ffn is not None:
+                s.ffn, s.experts, s.top, s.ff, s.limit = _lib.FFN_MOE, ffn.experts, ffn.top, ffn.ff, ffn.limit
+        return arr, keep
+
+
+class StackModel(DecoderModel):
+    """A decoder made of layer specs (``StackConfig``) over dense bf16 weights.
+
+    weights: name -> ``QuantLinear.from_bf16`` for ``embedding``, optional ``lm_head`` and
+    ``layers.{i}.{in,out}`` (the mixer's input projections as one weight: q | k | v, lightning
+    q | k | v | g) and ``layers.{i}.{gate,up,down,router}`` (the experts one after the other);
+    name -> f32 tensor for ``embed_norm``, ``final_norm``, ``layers.{i}.{norm1,norm2}`` and, in
+    lightning layers, ``layers.{i}.mix_norm``.  Logits are f32."""
+
+    LINEARS = {"in": 0, "out": 3, "gate": 4, "up": 5, "down": 6, "router": 7}
+    NORMS = {"norm1": 0, "norm2": 1, "mix_norm": 2}
+
+    def __init__(self, cfg: StackConfig, weights: dict, dtype: torch.dtype = torch.bfloat16, max_tokens: int = 512):
+        self.cfg, self.dtype, self.weights, self.tp = cfg, dtype, weights, None
+        self.max_tokens, self.logits_dtype = max_tokens, torch.float32
+        specs, _keep = cfg.c_specs()
+        c = _CConfig(n_layers=len(cfg.layers), d_model=cfg.d_model, vocab=cfg.vocab_size, max_seq=cfg.max_seq_len,
+                     rms_eps=cfg.rms_norm_eps, tied=1 if cfg.tie_embeddings else 0)
+        self._create(lib.ab2_model_create_stack, C.byref(c), specs, dtype_code(dtype), max_tokens)
+        for name, w in weights.items():
+            layer, leaf = -1, name
+            if name.startswith("layers."):
+                layer, leaf = int(name.split(".")[1]), name.split(".")[2]
+            if layer < 0 and leaf in ("embedding", "lm_head"):
+                check(lib.ab2_model_set_linear(self._h, -1, int(leaf == "lm_head"), w._h))
+            elif layer < 0:
+                self._norm(-1, int(leaf == "embed_norm"), w)
+            elif leaf in self.NORMS:
+                self._norm(layer, self.NORMS[leaf], w)
+            else:
+                check(lib.ab2_model_set_linear(self._h, layer, self.LINEARS[leaf], w._h))
+        check(lib.ab2_model_finalize(self._h))
+
+    @property
+    def kv_dtype(self) -> str:
+        return "f32" if self.dtype == torch.float32 else "bf16"
+
+    def empty_kv_cache_with_capacity(self, capacity: int, batch: int = 1, dtype: str | None = None) -> KVCache:
+        if dtype not in (None, self.kv_dtype):
+            raise _lib.Ab2Error(-3, f"this model caches {self.kv_dtype}, not {dtype}")
+        return KVCache.for_stack(self.cfg, capacity, batch, self.max_tokens, self.kv_dtype)
+
 
 class InferenceEngine:
     """Greedy generation from raw token ids, at model level: exactly
@@ -180,8 +308,8 @@ class InferenceEngine:
     token 0, crates/aarambh-studio-inference/src/engine.rs:898-911; ``eos_step``
     reports where it would have)."""
 
-    def __init__(self, model: AarambhModel, kv_dtype: str = "f32"):
-        self.model, self.kv_dtype = model, kv_dtype
+    def __init__(self, model: DecoderModel, kv_dtype: str | None = None):
+        self.model, self.kv_dtype = model, kv_dtype or model.kv_dtype
 
     def generate_from_token_ids(self, prompt_ids, max_new_tokens: int, eos_token_id: int = 0,
                                 on_device_sampling: bool = True):
@@ -195,7 +323,9 @@ class InferenceEngine:
         stream = torch.cuda.Stream()   # a capturable (non-default) stream for the graph-replayed steps
         stream.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(stream):
-            logits = m.forward_with_cache(prompt, 0, cache, last_only=True)
+            step = m.max_tokens        # a long prompt goes in as many portions as the workspace asks for
+            for off in range(0, P, step):
+                logits = m.forward_with_cache(prompt[:, off:off + step], off, cache, last_only=True)
             tokens = torch.empty(max_new_tokens, dtype=torch.int32, device="cuda")
             tokens[0:1] = argmax(logits.view(1, -1))
             if on_device_sampling:

@@ -57,6 +57,14 @@ class QuantLinear:
         return cls(h.value)
 
     @classmethod
+    def from_bf16(cls, weight: torch.Tensor):
+        """A dense bf16 weight [out_features, in_features] (host or device tensor), not quantised."""
+        if weight.dtype != torch.bfloat16 or weight.dim() != 2:
+            raise _lib.Ab2Error(-3, "from_bf16 expects a 2-D bfloat16 tensor")
+        weight = weight.contiguous()
+        return cls._make(lib.ab2_qweight_from_bf16, _ptr(weight), weight.shape[0], weight.shape[1])
+
+    @classmethod
     def from_i8_tensor(cls, codes, scale: float, N: int, K: int):
         codes = _contig(codes, np.int8)
         return cls._make(lib.ab2_qweight_from_i8_tensor, _ptr(codes), float(scale), N, K)
@@ -138,6 +146,10 @@ class QuantLinear:
         """Packed codes and parameters as numpy arrays (constructor layout)."""
         N, K, g = self.out_features, self.in_features, self.group
         n = N * K
+        if self.format == _lib.FMT_BF16:
+            codes = np.empty((N, K), np.uint16)
+            check(lib.ab2_qweight_export(self._h, codes.ctypes.data, None, None))
+            return codes, None, None
         if self.format == _lib.FMT_I8:
             codes = np.empty((N, K), np.int8); scales = np.empty(N, np.float32)
             check(lib.ab2_qweight_export(self._h, codes.ctypes.data, scales.ctypes.data, None))

@@ -20,7 +20,7 @@ import torch
 
 from . import _lib
 from .dispatch import argmax
-from .model import AarambhModel
+from .model import DecoderModel
 
 
 @dataclass
@@ -42,11 +42,59 @@ class SessionEngine:
     """Up to ``max_batch`` concurrent sessions over one model (the serving
     batcher's default is 8, prefill chunks of 128 tokens; batching.rs:35-52)."""
 
-    def __init__(self, model: AarambhModel, max_batch: int = 8, capacity: int | None = None, kv_dtype: str = "f32"):
+    def __init__(self, model: DecoderModel, max_batch: int = 8, capacity: int | None = None,
+                 kv_dtype: str | None = None):
         self.model = model
         self.capacity = capacity or model.cfg.max_seq_len
-        self.cache = model.empty_kv_cache_with_capacity(self.capacity, max_batch, kv_dtype)
+        self.cache = model.empty_kv_cache_with_capacity(self.capacity, max_batch, kv_dtype or model.kv_dtype)
         self.free_rows = list(range(max_batch))
+        self._step = None   # buffers and stream of the graph-replayed one-token feed
+
+    # -- rows of the cache -----------------------------------------------------
+    def open_row(self) -> int:
+        """An empty row for a new sequence."""
+        if not self.free_rows:
+            raise _lib.Ab2Error(-1, "every row of the batch holds a session")
+        row = self.free_rows.pop(0)
+        self.cache.truncate(0, row)
+        return row
+
+    def close_row(self, row: int) -> None:
+        """Gives a row back (its cached tokens and states are dropped)."""
+        self.cache.truncate(0, row)
+        self.free_rows.append(row)
+        self.free_rows.sort()
+
+    def feed(self, row: int, tokens, want=()) -> torch.Tensor:
+        """Runs given tokens through the model from where ``row`` stands and returns the logits
+        [len(want), vocab] at the places ``want`` (ascending) among them.  One token goes through the
+        graph-replayed decode step, more through prefill portions of at most the model's workspace."""
+        tokens, want = [int(t) for t in tokens], [int(w) for w in want]
+        if len(tokens) == 1:
+            logits = self._feed_one(row, tokens[0])
+            return logits[[0] * len(want)]
+        outs = []
+        for off in range(0, len(tokens), self.model.max_tokens):
+            part = torch.tensor([tokens[off:off + self.model.max_tokens]])
+            here = [w - off for w in want if off <= w < off + part.shape[1]]
+            if not here:
+                self.model.extend_cache(part, self.cache, row)
+                continue
+            logits = self.model.forward_with_cache(part, self.cache.seq_len(row), self.cache, row=row)[0]
+            outs.append(logits[here])
+        return torch.cat(outs) if outs else torch.empty((0, self.model.cfg.vocab_size), device="cuda")
+
+    def _feed_one(self, row: int, token: int) -> torch.Tensor:
+        if self._step is None:
+            self._step = (torch.cuda.Stream(), torch.empty(1, dtype=torch.int32, device="cuda"),
+                          torch.empty((1, self.model.cfg.vocab_size), dtype=self.model.logits_dtype, device="cuda"))
+        stream, ids, logits = self._step
+        stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(stream):
+            ids.fill_(token)
+            self.model.decode_step_rows(ids, [row], self.cache, logits, None)
+        torch.cuda.current_stream().wait_stream(stream)
+        return logits
 
     # -- engine.rs:271-318 ---------------------------------------------------
     def prepare_session_with_chunk_size(self, prompt_ids, max_new_tokens: int, chunk_size: int = 128,
@@ -59,10 +107,7 @@ class SessionEngine:
         max_seq = min(self.model.cfg.max_seq_len, self.capacity)
         if len(ids) >= max_seq:
             raise _lib.Ab2Error(-1, f"prompt has {len(ids)} tokens but model max_seq_len is {max_seq}")
-        if not self.free_rows:
-            raise _lib.Ab2Error(-1, "every row of the batch holds a session")
-        row = self.free_rows.pop(0)
-        self.cache.truncate(0, row)
+        row = self.open_row()
         logits = None
         for off in range(0, len(ids), chunk_size):
             chunk = torch.tensor([ids[off:off + chunk_size]])
@@ -109,28 +154,33 @@ class SessionEngine:
 
     def release(self, session: GenerationSession) -> None:
         """Gives the session's row back (its cached tokens are dropped)."""
-        self.cache.truncate(0, session.row)
-        self.free_rows.append(session.row)
-        self.free_rows.sort()
+        self.close_row(session.row)
         session.finished = True
 
 
-def verify_draft(model: AarambhModel, cache, row: int, base_len: int, pending_token: int, draft_tokens):
+def verify_draft(model: DecoderModel, cache, row: int, base_len: int, pending_token: int, draft_tokens):
     """Target-side round of greedy speculative decoding (speculative.rs:304-318,
     388-418): one forward of ``[pending_token] + draft_tokens`` against the cache
     at ``base_len``; draft token i is accepted while it equals the target's greedy
     choice after the tokens before it.  The cache row is left holding exactly the
     accepted prefix (an O(1) ``truncate`` where the reference restores a snapshot
-    and replays the accepted tokens).  Returns (number of accepted draft tokens,
+    and replays the accepted tokens; a cache with recurrent states does as the reference does).  Returns (number of accepted draft tokens,
     the target's next token after them, logits [1 + len(draft), vocab])."""
     draft = [int(t) for t in draft_tokens]
     if cache.seq_len(row) != base_len:
         raise _lib.Ab2Error(-1, f"cache row holds {cache.seq_len(row)} tokens, expected {base_len}")
+    if cache.has_state():
+        cache.save_row(row)
     ids = torch.tensor([[int(pending_token)] + draft])
     logits = model.forward_with_cache(ids, base_len, cache, row=row)[0]
     choice = argmax(logits).cpu().tolist()
     accepted = 0
     while accepted < len(draft) and choice[accepted] == draft[accepted]:
         accepted += 1
-    cache.truncate(base_len + 1 + accepted, row)
+    if cache.has_state() and accepted < len(draft):
+        # a recurrent state cannot be cut back: restore it and run the accepted tokens again
+        cache.truncate(base_len, row)
+        model.extend_cache(ids[:, :1 + accepted], cache, row)
+    else:
+        cache.truncate(base_len + 1 + accepted, row)
     return accepted, choice[accepted], logits

@@ -70,6 +70,8 @@ int ab2_device_status(int *status_host);
  * The packed bytes stay on the GPU; the reference instead dequantises to dense
  * f32 at load (crates/aarambh-studio-weights/src/gguf.rs:152-163,195-241). */
 
+/* A dense bf16 weight, not quantised (a layer stack's checkpoint format). */
+int ab2_qweight_from_bf16(ab2_qweight **out, const uint16_t *weight, int N, int K);
 /* I8QuantizedTensor, one scale per tensor
  * (crates/aarambh-studio-quant/src/absmax.rs:7-24, types.rs:66-75). */
 int ab2_qweight_from_i8_tensor(ab2_qweight **out, const int8_t *codes, float scale, int N, int K);
@@ -177,6 +179,35 @@ int ab2_argmax(const void *logits_dev, int rows, int vocab, ab2_dtype dtype, uin
 int ab2_embedding_forward(const ab2_qweight *table, const uint32_t *ids_dev, int tokens, void *out_dev,
                           ab2_dtype dtype, ab2_stream stream);
 
+/* ---- layer stacks ------------------------------------------------------------
+ * A decoder whose layers differ: each names its mixer (how tokens exchange
+ * information) and its feed-forward, with every constant as a parameter.  No
+ * counterpart in the reference, whose decoder repeats one block. */
+typedef enum {
+    AB2_MIX_ATTENTION = 0, /* grouped-query softmax attention over a sliding window */
+    AB2_MIX_LIGHTNING = 1  /* linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q */
+} ab2_mixer;
+typedef enum {
+    AB2_FFN_NONE = 0,
+    AB2_FFN_MOE = 1 /* mixture of experts: sigmoid scores, the score multiplies the expert's input, clamped gated unit */
+} ab2_ffn;
+typedef struct {
+    int mixer;          /* ab2_mixer */
+    int heads, dim, vdim;
+    int kv_heads;       /* attention */
+    int window;         /* attention: keys a query sees, itself included; 0 = all */
+    int rot_dims;       /* attention: leading dimensions that are rotated, pairs (2i, 2i + 1); 0 = none */
+    double rot_base;
+    int qk_norm;        /* attention: q and k divided by their root mean square after the rotation */
+    float scale;        /* attention: score = scale q.k */
+    int v_mix;          /* attention: values are mixed with those of the stack's first layer that has this set */
+    float v_lambda;     /* their weight: v <- (1 - lambda) v + lambda v_first */
+    const float *decay; /* lightning: [heads], host memory, copied by the calls that take a spec */
+    int ffn;            /* ab2_ffn */
+    int experts, top, ff;
+    float limit;        /* clamp of the gated unit */
+} ab2_layer_spec;
+
 /* ---- KV cache --------------------------------------------------------------
  * KVCache with preallocated storage (crates/aarambh-studio-nn/src/kvcache.rs:
  * 236-369) for `batch` independent sequences; INT8 storage quantises every
@@ -189,6 +220,18 @@ int ab2_embedding_forward(const ab2_qweight *table, const uint32_t *ids_dev, int
 int ab2_kv_create(ab2_kv **out, int n_layers, int batch, int capacity, int kv_heads, int head_dim,
                   int n_heads, ab2_kv_dtype dtype);
 int ab2_kv_destroy(ab2_kv *kv);
+/* The cache of a layer stack for `batch` sequences of at most `capacity` tokens: an attention layer
+ * keeps the last window - 1 + max_step keys and values (position p in slot p mod that), a recurrent
+ * layer one f32 state per sequence.  max_step is the most tokens one forward call appends to a row.
+ * dtype is AB2_KV_F32 or AB2_KV_BF16 and equals the model's activation type.
+ * ab2_kv_{truncate,clear,seq_len,capacity,clone,destroy} apply; the tensors are written by the model's steps. */
+int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n_layers, int batch, int capacity,
+                        int max_step, ab2_kv_dtype dtype);
+/* A recurrent state cannot be cut back: ab2_kv_save_row remembers the row at its current length, and
+ * ab2_kv_truncate to that length restores it (a row is otherwise cut to 0 only).  On caches without
+ * recurrent layers it does nothing. */
+int ab2_kv_save_row(ab2_kv *kv, int row, ab2_stream stream);
+int ab2_kv_has_state(const ab2_kv *kv, int *has_state);
 /* KVCache::update (kvcache.rs:335-368) for a single-layer cache: k, v
  * [nrows, S, kv_heads, head_dim] of element type `dtype` are appended to rows
  * row0..row0+nrows-1 at their current lengths, which then grow by S.
@@ -282,6 +325,22 @@ int ab2_model_set_norm(ab2_model *m, int layer, int which, const float *weight);
  * workspace. */
 int ab2_model_finalize(ab2_model *m);
 int ab2_model_rope_tables(const ab2_model *m, const float **cos_dev, const float **sin_dev);
+
+/* A decoder made of `n_layers` layer specs over one residual stream, which is kept in f32 whatever
+ * `dtype` is (AB2_F32 or AB2_BF16): x = RMSNorm(embedding[token]); per layer x += RMSNorm(mixer(x)),
+ * then x += RMSNorm(ffn(x)) where the layer has a feed-forward; logits = head . RMSNorm(x).  Of cfg
+ * d_model, vocab, max_seq, rms_eps and tied are read.  Logits are f32.
+ * Weights (FMT bf16, ab2_qweight_from_bf16) by ab2_model_set_linear, layer >= 0:
+ *   which = 0  the mixer's input projections as one weight: attention q | k | v rows, lightning q | k | v | g rows
+ *   which = 3  the mixer's output projection
+ *   which = 4, 5, 6  the experts' gate, up ([experts * ff, d_model]) and down ([experts * d_model, ff]), expert by expert
+ *   which = 7  the router [experts, d_model]
+ * Norms by ab2_model_set_norm, layer >= 0: which = 0 after the mixer, 1 after the feed-forward, 2 the lightning
+ * mixer's own over heads * vdim; layer < 0: which = 0 the final norm, 1 the embedding's.
+ * The handle then serves ab2_model_finalize, ab2_model_forward*, ab2_model_decode_step* with caches of
+ * ab2_kv_create_stack; offsets must be the cache lengths. */
+int ab2_model_create_stack(ab2_model **out, const ab2_model_config *cfg, const ab2_layer_spec *specs, ab2_dtype dtype,
+                           int max_tokens);
 
 /* ---- tensor parallelism ------------------------------------------------------
  * Megatron-style sharding of the decoder over the GPUs of one box, one process

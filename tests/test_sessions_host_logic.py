@@ -23,6 +23,9 @@ class FakeCache:
     def seq_len(self, row=0):
         return self.lens[row]
 
+    def has_state(self):
+        return False
+
 
 class FakeModel:
     """Logits put the maximum at (last token + 1) % vocab; every call is recorded."""
@@ -30,6 +33,9 @@ class FakeModel:
     class Cfg:
         max_seq_len = 64
         vocab_size = 32
+
+    kv_dtype = "f32"
+    max_tokens = 64
 
     def __init__(self):
         self.cfg = self.Cfg()
