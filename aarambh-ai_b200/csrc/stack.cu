@@ -287,16 +287,30 @@ static int lightning_mixer(Stack *st, StackLayer &L, ab2_kv *kv, int layer, int 
     return launch_residual_norm(n, RN_GATED, nrows * S, st->dtype, s);
 }
 
-static int moe_ffn(Stack *st, StackLayer &L, const void *in, int T, cudaStream_t s) {
-    const ab2_layer_spec &sp = L.spec;
+// Scratch of a mixture of experts.
+struct MoeScratch {
+    float *router_z;       // [T][experts]
+    int *route_int;        // 2 T top + 2 (experts + 1)
+    float *route_score;    // [T top]
+    void *act, *gathered;  // [T top][ff], [T top][width] in the activation type
+};
+
+// parts[t * top + slot] = W_down glu(s W_gate x_t, s W_up x_t) of the token's slot-th expert, f32
+static int moe_experts(const ab2_layer_spec &sp, const ab2_qweight *router, const ab2_qweight *gate, const ab2_qweight *up,
+                       const ab2_qweight *down, const void *in, int T, ab2_dtype dtype, const MoeScratch &w, float *parts, cudaStream_t s) {
     MoeRoute r = {};
     r.E = sp.experts; r.top = sp.top; r.pairs = T * sp.top;
-    r.perm = st->route_int; r.expert = r.perm + r.pairs; r.offset = r.expert + r.pairs; r.active = r.offset + sp.experts + 1;
-    r.score = st->route_score;
-    STEP(linear_bf16(L.router, in, T, st->dtype, st->router_z, LIN_F32, 0, s));
-    STEP(moe_route(st->router_z, T, r, s));
-    STEP(linear_moe_glu(L.gate, L.up, in, st->dtype, st->act, sp.limit, r, st->gathered, s));
-    return linear_moe_down(L.down, st->act, st->dtype, st->parts, r, s);
+    r.perm = w.route_int; r.expert = r.perm + r.pairs; r.offset = r.expert + r.pairs; r.active = r.offset + sp.experts + 1;
+    r.score = w.route_score;
+    STEP(linear_bf16(router, in, T, dtype, w.router_z, LIN_F32, 0, s));
+    STEP(moe_route(w.router_z, T, r, s));
+    STEP(linear_moe_glu(gate, up, in, dtype, w.act, sp.limit, r, w.gathered, s));
+    return linear_moe_down(down, w.act, dtype, parts, r, s);
+}
+
+static int moe_ffn(Stack *st, StackLayer &L, const void *in, int T, cudaStream_t s) {
+    const MoeScratch w = {st->router_z, st->route_int, st->route_score, st->act, st->gathered};
+    return moe_experts(L.spec, L.router, L.gate, L.up, L.down, in, T, st->dtype, w, st->parts, s);
 }
 
 int stack_forward(Stack *st, ab2_kv *kv, const uint32_t *ids, int S, int row0, int nrows, int logits_mode, float *logits,
@@ -342,3 +356,91 @@ int stack_forward(Stack *st, ab2_kv *kv, const uint32_t *ids, int S, int row0, i
 }
 
 }  // namespace ab2
+
+// ---- the mechanisms as operators of their own ---------------------------------------
+
+static int check_mixer_call(const ab2_kv *kv, int layer, const ab2_layer_spec *spec, int mixer, const void *qkv, const void *out, int S,
+                            int row0, int nrows, ab2_dtype dtype) {
+    AB2_REQUIRE(kv && spec && qkv && out, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(kv->layers && layer >= 0 && layer < kv->L, AB2_ERR_BAD_SHAPE, "layer %d of a stack cache expected", layer);
+    AB2_REQUIRE(spec->mixer == mixer, AB2_ERR_BAD_ARG, "the spec names another mixer");
+    if (mixer == AB2_MIX_ATTENTION) STEP(check_spec(*spec, layer));
+    const KvLayer &l = kv->layers[layer];
+    const bool rec = mixer == AB2_MIX_LIGHTNING;
+    AB2_REQUIRE(l.recurrent == rec && l.kvh == (rec ? spec->heads : spec->kv_heads) && l.kd == spec->dim && l.vd == spec->vdim,
+                AB2_ERR_BAD_SHAPE, "cache layer %d does not match the spec", layer);
+    AB2_REQUIRE(dtype == AB2_F32 || dtype == AB2_BF16, AB2_ERR_BAD_DTYPE, "unsupported dtype %d", (int)dtype);
+    AB2_REQUIRE(kv->dtype == (dtype == AB2_F32 ? AB2_KV_F32 : AB2_KV_BF16), AB2_ERR_BAD_DTYPE, "the cache's type differs from the activations'");
+    AB2_REQUIRE(S > 0 && nrows > 0 && row0 >= 0 && row0 + nrows <= kv->B && (long long)nrows * S <= 65535, AB2_ERR_BAD_SHAPE,
+                "rows %d..%d of %d tokens do not fit", row0, row0 + nrows, S);
+    AB2_REQUIRE(rec || l.cap == kv->cap || l.window - 1 + S <= l.cap, AB2_ERR_CAPACITY, "a step of %d tokens exceeds what the cache was made for", S);
+    for (int i = 0; i < nrows; ++i)
+        AB2_REQUIRE(kv->lens_host[row0 + i] + S <= kv->cap, AB2_ERR_CAPACITY, "KV cache length %d exceeds capacity %d", kv->lens_host[row0 + i] + S, kv->cap);
+    return AB2_OK;
+}
+
+AB2_API int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *qkv_dev, void *v_first_dev, int v_mode,
+                                 const float *cos_dev, const float *sin_dev, float eps, void *out_dev, int S, int row0, int nrows,
+                                 ab2_dtype dtype, ab2_stream stream) {
+    STEP(check_mixer_call(kv, layer, spec, AB2_MIX_ATTENTION, qkv_dev, out_dev, S, row0, nrows, dtype));
+    AB2_REQUIRE(spec->rot_dims == 0 || (cos_dev && sin_dev), AB2_ERR_BAD_ARG, "null rotation tables");
+    AB2_REQUIRE(v_mode >= 0 && v_mode <= 2 && (v_mode == 0 || v_first_dev), AB2_ERR_BAD_ARG, "value mixing %d needs the first values", v_mode);
+    WindowPrepArgs p = {};
+    p.kv = kv_layer_view(kv, layer);
+    p.qkv = qkv_dev; p.stride = (long long)(spec->heads + spec->kv_heads) * spec->dim + (long long)spec->kv_heads * spec->vdim;
+    p.S = S; p.row0 = row0; p.H = spec->heads; p.G = spec->kv_heads; p.dim = spec->dim; p.vdim = spec->vdim;
+    p.rot_dims = spec->rot_dims; p.qk_norm = spec->qk_norm; p.cos_t = cos_dev; p.sin_t = sin_dev; p.eps = eps;
+    p.v_first = v_first_dev; p.v_mode = v_mode; p.lambda = spec->v_lambda;
+    STEP(window_prep(p, nrows, dtype, (cudaStream_t)stream));
+    WindowAttnArgs a = {};
+    a.kv = p.kv; a.q = qkv_dev; a.q_stride = p.stride; a.out = out_dev; a.S = S; a.row0 = row0; a.H = spec->heads;
+    a.rep = spec->heads / spec->kv_heads; a.dim = spec->dim; a.vdim = spec->vdim; a.scale = spec->scale;
+    int max_len = 0;
+    for (int i = 0; i < nrows; ++i) max_len = std::max(max_len, kv->lens_host[row0 + i] + S);
+    return window_attention(kv, a, nrows, max_len, dtype, (cudaStream_t)stream);
+}
+
+AB2_API int ab2_lightning_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, const float *decay_pow_dev, const void *qkv_dev,
+                                    long long stride, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream) {
+    STEP(check_mixer_call(kv, layer, spec, AB2_MIX_LIGHTNING, qkv_dev, out_dev, S, row0, nrows, dtype));
+    AB2_REQUIRE(decay_pow_dev != nullptr, AB2_ERR_BAD_ARG, "null decay table");
+    AB2_REQUIRE(stride >= (long long)spec->heads * (2 * spec->dim + spec->vdim), AB2_ERR_BAD_SHAPE, "row stride %lld is too short", stride);
+    LightningArgs a = {};
+    a.kv = kv_layer_view(kv, layer);
+    a.qkv = qkv_dev; a.stride = stride; a.out = out_dev; a.S = S; a.row0 = row0; a.H = spec->heads; a.dim = spec->dim; a.vdim = spec->vdim;
+    a.decay_pow = decay_pow_dev;
+    return lightning_attention(a, nrows, dtype, (cudaStream_t)stream);
+}
+
+static size_t up256(size_t n) { return (n + 255) / 256 * 256; }
+
+AB2_API int ab2_moe_workspace(const ab2_layer_spec *spec, int width, int tokens, ab2_dtype dtype, size_t *bytes) {
+    AB2_REQUIRE(spec && bytes, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(width > 0 && tokens > 0 && spec->experts > 0 && spec->top > 0 && spec->ff > 0, AB2_ERR_BAD_SHAPE, "sizes must be positive");
+    const size_t P = (size_t)tokens * spec->top, esz = dtype_size(dtype);
+    *bytes = up256((size_t)tokens * spec->experts * 4) + up256((2 * P + 2 * (spec->experts + 1)) * 4) + up256(P * 4) + up256(P * spec->ff * esz) +
+             up256(P * width * esz);
+    return AB2_OK;
+}
+
+AB2_API int ab2_moe_forward(const ab2_layer_spec *spec, const ab2_qweight *router, const ab2_qweight *gate, const ab2_qweight *up,
+                            const ab2_qweight *down, const void *x_dev, int tokens, ab2_dtype dtype, float *parts_dev, void *workspace_dev,
+                            ab2_stream stream) {
+    AB2_REQUIRE(spec && router && gate && up && down && x_dev && parts_dev && workspace_dev, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(tokens > 0 && spec->experts > 0 && spec->experts <= 1024 && spec->top > 0 && spec->top <= spec->experts && spec->ff > 0,
+                AB2_ERR_BAD_SHAPE, "%d of %d experts of width %d over %d tokens", spec->top, spec->experts, spec->ff, tokens);
+    AB2_REQUIRE(dtype == AB2_F32 || dtype == AB2_BF16, AB2_ERR_BAD_DTYPE, "unsupported dtype %d", (int)dtype);
+    const int E = spec->experts, d = router->K;
+    for (const ab2_qweight *w : {router, gate, up, down}) AB2_REQUIRE(w->fmt == FMT_BF16, AB2_ERR_UNSUPPORTED, "experts are dense bf16 weights");
+    AB2_REQUIRE(router->N == E && gate->N == E * spec->ff && up->N == gate->N && gate->K == d && up->K == d && down->N == E * d && down->K == spec->ff,
+                AB2_ERR_BAD_SHAPE, "the experts' weights do not match the spec");
+    const size_t P = (size_t)tokens * spec->top, esz = dtype_size(dtype);
+    char *p = (char *)workspace_dev;
+    MoeScratch w;
+    w.router_z = (float *)p; p += up256((size_t)tokens * E * 4);
+    w.route_int = (int *)p; p += up256((2 * P + 2 * (E + 1)) * 4);
+    w.route_score = (float *)p; p += up256(P * 4);
+    w.act = p; p += up256(P * spec->ff * esz);
+    w.gathered = p;
+    return moe_experts(*spec, router, gate, up, down, x_dev, tokens, dtype, w, parts_dev, (cudaStream_t)stream);
+}

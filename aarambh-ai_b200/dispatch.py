@@ -5,6 +5,8 @@ allocated, inputs are borrowed, tensors must be CUDA and are made contiguous.
 """
 from __future__ import annotations
 
+import ctypes as C
+
 import torch
 
 from . import _lib
@@ -122,3 +124,68 @@ def embedding_forward(table, ids: torch.Tensor, dtype: torch.dtype) -> torch.Ten
     check(lib.ab2_embedding_forward(table._h, ids.data_ptr(), ids.numel(), out.data_ptr(), dtype_code(dtype),
                                     stream_ptr()))
     return out
+
+
+# -- mechanisms of layer stacks (``model.StackConfig``), one layer of a stack cache at a time --------
+
+def rotation_tables(positions: int, dims: int, base: float):
+    """cos, sin [positions, dims / 2] (f32) of position * base ** (-2i / dims), the angles in f64."""
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    a = torch.arange(positions, dtype=torch.float64)[:, None] * f
+    return a.cos().float().cuda(), a.sin().float().cuda()
+
+
+def decay_powers(decay) -> torch.Tensor:
+    """[heads, 65] f32: powers 0..64 of every head's decay."""
+    d = torch.tensor(list(decay), dtype=torch.float64)[:, None]
+    return torch.pow(d, torch.arange(65, dtype=torch.float64)).float().cuda().contiguous()
+
+
+def window_attention(cache, cfg, layer: int, qkv: torch.Tensor, tables, eps: float, v_first=None, v_mode: int = 0,
+                     row0: int = 0) -> torch.Tensor:
+    """qkv [rows, S, heads dim + kv_heads dim + kv_heads vdim] (overwritten) -> [rows, S, heads vdim]."""
+    qkv = _cuda(qkv, "qkv")
+    specs, _keep = cfg.c_specs()
+    sp = specs[layer]
+    rows, S = qkv.shape[:2]
+    out = torch.empty((rows, S, sp.heads * sp.vdim), dtype=qkv.dtype, device=qkv.device)
+    cos, sin = tables if tables is not None else (None, None)
+    check(lib.ab2_window_attention(cache._h, layer, C.byref(sp), qkv.data_ptr(), v_first.data_ptr() if v_first is not None else None,
+                                   v_mode, cos.data_ptr() if cos is not None else None, sin.data_ptr() if sin is not None else None,
+                                   float(eps), out.data_ptr(), S, row0, rows, dtype_code(qkv.dtype), stream_ptr()))
+    return out
+
+
+def lightning_attention(cache, cfg, layer: int, qkv: torch.Tensor, powers: torch.Tensor, row0: int = 0) -> torch.Tensor:
+    """qkv [rows, S, stride] starting with heads dim | heads dim | heads vdim -> f32 [rows, S, heads vdim]."""
+    qkv = _cuda(qkv, "qkv")
+    specs, _keep = cfg.c_specs()
+    sp = specs[layer]
+    rows, S, stride = qkv.shape
+    out = torch.empty((rows, S, sp.heads * sp.vdim), dtype=torch.float32, device=qkv.device)
+    check(lib.ab2_lightning_attention(cache._h, layer, C.byref(sp), powers.data_ptr(), qkv.data_ptr(), stride, out.data_ptr(), S, row0,
+                                      rows, dtype_code(qkv.dtype), stream_ptr()))
+    return out
+
+
+class MoeExperts:
+    """The feed-forward of ``model.MoeFfn`` over dense bf16 weights: x [tokens, width] -> the chosen
+    experts' outputs [tokens, top, width] (f32; their sum is the layer's output)."""
+
+    def __init__(self, ffn, router, gate, up, down):
+        self.spec = _lib.LayerSpec(ffn=_lib.FFN_MOE, experts=ffn.experts, top=ffn.top, ff=ffn.ff, limit=ffn.limit)
+        self.router, self.gate, self.up, self.down = router, gate, up, down
+        self._work = None
+
+    def __call__(self, x: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+        x = _cuda(x, "x")
+        T, width = x.shape
+        n = C.c_size_t()
+        check(lib.ab2_moe_workspace(C.byref(self.spec), width, T, dtype_code(x.dtype), C.byref(n)))
+        if self._work is None or self._work.numel() < n.value:
+            self._work = torch.empty(n.value, dtype=torch.uint8, device=x.device)
+        if out is None:
+            out = torch.empty((T, self.spec.top, width), dtype=torch.float32, device=x.device)
+        check(lib.ab2_moe_forward(C.byref(self.spec), self.router._h, self.gate._h, self.up._h, self.down._h, x.data_ptr(), T,
+                                  dtype_code(x.dtype), out.data_ptr(), self._work.data_ptr(), stream_ptr()))
+        return out

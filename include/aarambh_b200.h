@@ -264,6 +264,27 @@ int ab2_kv_clone(ab2_kv **out, const ab2_kv *src, ab2_stream stream);
 int ab2_kv_read(const ab2_kv *kv, int layer, int row, float *k_out_dev, float *v_out_dev,
                 ab2_stream stream);
 
+/* ---- mechanisms of layer stacks as operators ---------------------------------------
+ * Each works on one layer of a stack cache at the rows' current lengths, which it does not advance
+ * (ab2_kv_commit does, once every layer has run).
+ * Window attention: qkv_dev [nrows * S][heads dim | kv_heads dim | kv_heads vdim], the queries are
+ * rewritten; rotation and normalisation as the spec says (tables [positions][rot_dims / 2]); v_mode 1
+ * copies the values to v_first_dev [nrows * S][kv_heads vdim], 2 mixes them with it; out_dev
+ * [nrows * S][heads vdim]. */
+int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *qkv_dev, void *v_first_dev, int v_mode,
+                         const float *cos_dev, const float *sin_dev, float eps, void *out_dev, int S, int row0, int nrows,
+                         ab2_dtype dtype, ab2_stream stream);
+/* Lightning attention: rows of qkv_dev hold q, k (heads dim each) and v (heads vdim), `stride` elements
+ * apart; decay_pow_dev [heads][65] holds the powers 0..64 of each head's decay; out_dev [nrows * S][heads vdim] f32. */
+int ab2_lightning_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, const float *decay_pow_dev, const void *qkv_dev,
+                            long long stride, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
+/* Mixture of experts: parts_dev [tokens][top][width] f32, the chosen experts' outputs (their sum is the
+ * layer's).  Weights as in ab2_model_create_stack; workspace_dev holds ab2_moe_workspace bytes. */
+int ab2_moe_workspace(const ab2_layer_spec *spec, int width, int tokens, ab2_dtype dtype, size_t *bytes);
+int ab2_moe_forward(const ab2_layer_spec *spec, const ab2_qweight *router, const ab2_qweight *gate, const ab2_qweight *up,
+                    const ab2_qweight *down, const void *x_dev, int tokens, ab2_dtype dtype, float *parts_dev, void *workspace_dev,
+                    ab2_stream stream);
+
 /* ---- attention --------------------------------------------------------------
  * GroupedQueryAttention::forward_decode_batch attention step
  * (crates/aarambh-studio-nn/src/attention.rs:265-283 -> dispatch::
