@@ -414,6 +414,199 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
     }
 }
 
+// ---------------------------------------------------------------------------
+// Decode in bf16: one query per sequence.  The (up to 16) query heads of a KV head are the rows of
+// the MMA, the keys its columns.  grid (nsplit, G * head groups, rows), 4 warps: a CTA takes one of
+// nsplit runs of the visible keys and its warps deal them out 16 at a time; a warp streams its keys and
+// values through a ring of its own in shared memory (cp.async, no CTA barrier in the loop).  The warps
+// meet in shared memory at the end, the splits in window_merge_kernel.
+// ---------------------------------------------------------------------------
+constexpr int WD_STAGES = 3;
+
+template <int DP, int VP>
+__global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a) {
+    extern __shared__ __align__(1024) uint8_t smem[];
+    constexpr int KB = 16 * DP * 2, VB = 16 * VP * 2, STAGE = KB + VB;
+    __shared__ float wm[4][16], wl[4][16];
+    pdl_wait();
+    pdl_launch_dependents();
+    const KvLayer &l = a.kv.l;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+    const int groups = (a.rep + 15) / 16, kvh = blockIdx.y / groups, hg = blockIdx.y % groups;
+    const int head0 = kvh * a.rep + hg * 16, nh = min(16, a.rep - hg * 16);
+    const int rrow = blockIdx.z, row = kv_row(a.kv, a.row0, rrow);
+    const int pos = a.kv.lens[row], lo = max(0, pos - l.window + 1), n = pos + 1 - lo;
+    const int per = ((n + a.nsplit - 1) / a.nsplit + 63) & ~63;
+    const int j0 = lo + (int)blockIdx.x * per, j1 = min(pos + 1, j0 + per);
+    const __nv_bfloat16 *kb = (const __nv_bfloat16 *)l.k + ((size_t)row * l.kvh + kvh) * l.cap * l.kds;
+    const __nv_bfloat16 *vb = (const __nv_bfloat16 *)l.v + ((size_t)row * l.kvh + kvh) * l.cap * l.vds;
+    const uint32_t ring = (uint32_t)__cvta_generic_to_shared(smem) + warp * WD_STAGES * STAGE;
+
+    auto load = [&](int base, int st) {
+        if (base < j1) {
+            const uint32_t ks = ring + st * STAGE, vs = ks + KB;
+            const int slot0 = base % l.cap;
+#pragma unroll
+            for (int i = 0; i < 16 * (DP / 8) / 32; ++i) {
+                const int idx = lane + 32 * i, r = idx / (DP / 8), ch = idx % (DP / 8);
+                int slot = slot0 + min(r, j1 - 1 - base);  // keys past the run repeat its last (masked below)
+                if (slot >= l.cap) slot -= l.cap;
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(ks + r * DP * 2 + ((ch ^ (r & 7)) << 4)),
+                             "l"(kb + (size_t)slot * l.kds + (ch * 8 < l.kds ? ch * 8 : 0)), "r"(ch * 8 < l.kds ? 16 : 0));
+            }
+#pragma unroll
+            for (int i = 0; i < 16 * (VP / 8) / 32; ++i) {
+                const int idx = lane + 32 * i, r = idx / (VP / 8), ch = idx % (VP / 8);
+                int slot = slot0 + min(r, j1 - 1 - base);
+                if (slot >= l.cap) slot -= l.cap;
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(vs + r * VP * 2 + ((ch ^ (r & 7)) << 4)),
+                             "l"(vb + (size_t)slot * l.vds + (ch * 8 < l.vds ? ch * 8 : 0)), "r"(ch * 8 < l.vds ? 16 : 0));
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::);  // one group per stage, also an empty one
+    };
+#pragma unroll
+    for (int st = 0; st < WD_STAGES - 1; ++st) load(j0 + (st * 4 + warp) * 16, st);
+
+    uint32_t qf[DP / 16][4];
+    {
+        const __nv_bfloat16 *ra = (const __nv_bfloat16 *)a.q + (size_t)rrow * a.q_stride + (size_t)(head0 + min(g, nh - 1)) * a.dim;
+        const __nv_bfloat16 *rb = (const __nv_bfloat16 *)a.q + (size_t)rrow * a.q_stride + (size_t)(head0 + min(g + 8, nh - 1)) * a.dim;
+#pragma unroll
+        for (int ks = 0; ks < DP / 16; ++ks)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int d = ks * 16 + h * 8 + 2 * c;
+                const bool in = d < a.dim;
+                qf[ks][2 * h] = in ? *reinterpret_cast<const uint32_t *>(ra + d) : 0u;
+                qf[ks][2 * h + 1] = in ? *reinterpret_cast<const uint32_t *>(rb + d) : 0u;
+            }
+    }
+    const float sl = a.scale * 1.44269504088896341f;  // scores in powers of two
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f}, o[VP / 8][4];
+#pragma unroll
+    for (int i = 0; i < VP / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+
+    int st = 0;
+    for (int base = j0 + warp * 16; base < j1; base += 64) {
+        load(base + (WD_STAGES - 1) * 64, (st + WD_STAGES - 1) % WD_STAGES);
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(WD_STAGES - 1) : "memory");
+        __syncwarp();
+        const uint32_t ks0 = ring + st * STAGE, vs0 = ks0 + KB;
+        float s[2][4], bm[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s[nt][j] = 0.f;
+            const int r = nt * 8 + (lane & 7);
+#pragma unroll
+            for (int k2 = 0; k2 < DP / 32; ++k2) {
+                uint32_t b0, b1, b2, b3;
+                const uint32_t addr = ks0 + r * DP * 2 + (((k2 * 4 + (lane >> 3)) ^ (r & 7)) << 4);
+                asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                             : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3) : "r"(addr));
+                mma_bf16(s[nt], qf[2 * k2], b0, b1);
+                mma_bf16(s[nt], qf[2 * k2 + 1], b2, b3);
+            }
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                s[nt][j] = base + nt * 8 + 2 * c + (j & 1) < j1 ? s[nt][j] * sl : -INFINITY;
+                bm[j >> 1] = fmaxf(bm[j >> 1], s[nt][j]);
+            }
+        }
+        float corr[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {  // every 16 keys hold at least one of the run: the maximum is finite
+            bm[h] = fmaxf(bm[h], __shfl_xor_sync(0xffffffffu, bm[h], 1));
+            bm[h] = fmaxf(bm[h], __shfl_xor_sync(0xffffffffu, bm[h], 2));
+            const float m_new = fmaxf(m_run[h], bm[h]);
+            corr[h] = exp2f(m_run[h] - m_new);
+            m_run[h] = m_new;
+            l_run[h] *= corr[h];
+        }
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                s[nt][j] = exp2f(s[nt][j] - m_run[j >> 1]);
+                l_run[j >> 1] += s[nt][j];
+            }
+        uint32_t hi[4], lw[4];
+        split_pair(s[0][0], s[0][1], hi[0], lw[0]);
+        split_pair(s[0][2], s[0][3], hi[1], lw[1]);
+        split_pair(s[1][0], s[1][1], hi[2], lw[2]);
+        split_pair(s[1][2], s[1][3], hi[3], lw[3]);
+#pragma unroll
+        for (int i = 0; i < VP / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+        const int r = lane & 15;
+#pragma unroll
+        for (int vv = 0; vv < VP / 16; ++vv) {
+            uint32_t b0, b1, b2, b3;
+            const uint32_t addr = vs0 + r * VP * 2 + (((vv * 2 + (lane >> 4)) ^ (r & 7)) << 4);
+            asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+                         : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3) : "r"(addr));
+            mma_bf16(o[2 * vv], hi, b0, b1);
+            mma_bf16(o[2 * vv], lw, b0, b1);
+            mma_bf16(o[2 * vv + 1], hi, b2, b3);
+            mma_bf16(o[2 * vv + 1], lw, b2, b3);
+        }
+        // The products above have consumed every matrix load of this stage (a tensor-core instruction
+        // waits for its operands), so the refill two statements into the next pass cannot overtake them.
+        __syncwarp();
+        st = (st + 1) % WD_STAGES;
+    }
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
+        if (c == 0) { wm[warp][g + 8 * h] = m_run[h]; wl[warp][g + 8 * h] = l_run[h]; }
+    }
+    __syncthreads();  // the rings are free: they take the warps' sums, [4][16][VP] floats
+    float *wacc = reinterpret_cast<float *>(smem);
+#pragma unroll
+    for (int i = 0; i < VP / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) wacc[((size_t)warp * 16 + g + 8 * (j >> 1)) * VP + i * 8 + 2 * c + (j & 1)] = o[i][j];
+    __syncthreads();
+    for (int i = threadIdx.x; i < nh * a.vdim; i += 128) {
+        const int hh = i / a.vdim, d = i % a.vdim;
+        const float M = fmaxf(fmaxf(wm[0][hh], wm[1][hh]), fmaxf(wm[2][hh], wm[3][hh]));
+        float L = 0.f, A = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+            const float e = wm[w][hh] == -INFINITY ? 0.f : exp2f(wm[w][hh] - M);
+            L += e * wl[w][hh];
+            A += e * wacc[((size_t)w * 16 + hh) * VP + d];
+        }
+        const int head = head0 + hh;
+        if (a.nsplit == 1) {
+            ((__nv_bfloat16 *)a.out)[((size_t)rrow * a.H + head) * a.vdim + d] = __float2bfloat16_rn(A / L);
+        } else {
+            const size_t pi = ((size_t)rrow * a.H + head) * a.nsplit + blockIdx.x;
+            a.part_acc[pi * a.vdim + d] = A;
+            // the merge works in natural exponents
+            if (d == 0) { a.part_ml[pi * 2] = M * 0.693147180559945309f; a.part_ml[pi * 2 + 1] = L; }
+        }
+    }
+}
+
+template <int DP, int VP>
+cudaError_t launch_decode(const WindowAttnArgs &a, dim3 grid, cudaStream_t s) {
+    constexpr int smem = 4 * WD_STAGES * 16 * (DP + VP) * 2 > 4 * 16 * VP * 4 ? 4 * WD_STAGES * 16 * (DP + VP) * 2 : 4 * 16 * VP * 4;
+    static bool configured[64] = {false};
+    int dev = 0;
+    cudaGetDevice(&dev);
+    if (dev >= 0 && dev < 64 && !configured[dev]) {
+        cudaError_t e = cudaFuncSetAttribute(window_decode_mma_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return e;
+        configured[dev] = true;
+    }
+    return launch_kernel(window_decode_mma_kernel<DP, VP>, grid, dim3(128), (size_t)smem, s, a);
+}
+
 template <typename T, int REP>
 cudaError_t launch_simt(const WindowAttnArgs &a, dim3 grid, size_t smem, cudaStream_t s) {
     if (a.vdim <= 32) return launch_kernel(window_attn_kernel<T, REP, 1>, grid, dim3(128), smem, s, a);
@@ -440,9 +633,23 @@ template <typename T>
 int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cudaStream_t s) {
     cudaError_t e;
     const KvLayer &l = a.kv.l;
-    if (sizeof(T) == 2 && a.S >= 16 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 128 && a.vdim <= 128 && a.q_stride % 2 == 0) {
+    const bool on_mma = sizeof(T) == 2 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 128 && a.vdim <= 128 && a.q_stride % 2 == 0;
+    if (on_mma && a.S >= 16) {
         if (a.dim <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, nrows, s) : launch_mma<64, 128>(a, nrows, s);
         else e = a.vdim <= 64 ? launch_mma<128, 64>(a, nrows, s) : launch_mma<128, 128>(a, nrows, s);
+        if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window attention launch failed: %s", cudaGetErrorString(e));
+        return AB2_OK;
+    }
+    if (on_mma && a.S == 1) {
+        const int units = l.kvh * ((a.rep + 15) / 16) * nrows, reach = std::min(l.window, max_len);
+        // two CTAs per SM hold the streams that cover HBM's latency; a split keeps at least 128 keys
+        const int want = (2 * device_sm_count() + units - 1) / units;
+        a.nsplit = std::max(1, std::min(std::min(want, (reach + 127) / 128), kv->max_splits));
+        const dim3 grid(a.nsplit, l.kvh * ((a.rep + 15) / 16), nrows);
+        if (a.dim <= 64) e = a.vdim <= 64 ? launch_decode<64, 64>(a, grid, s) : launch_decode<64, 128>(a, grid, s);
+        else e = a.vdim <= 64 ? launch_decode<128, 64>(a, grid, s) : launch_decode<128, 128>(a, grid, s);
+        if (e == cudaSuccess && a.nsplit > 1)
+            e = launch_kernel(window_merge_kernel<T>, dim3(a.H, nrows), dim3(std::min(128, (a.vdim + 31) / 32 * 32)), 0, s, a);
         if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window attention launch failed: %s", cudaGetErrorString(e));
         return AB2_OK;
     }

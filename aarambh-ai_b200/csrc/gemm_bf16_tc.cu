@@ -22,6 +22,7 @@
 #include <cuda.h>
 
 #include <algorithm>
+#include <cmath>
 
 #include "linear_bf16.cuh"
 #include "tcgen05_util.cuh"
@@ -216,8 +217,8 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                         : "r"(taddr));
                 }
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-                if (n >= a.N) continue;
                 if (MODE == LIN_DENSE) {
+                    if (n >= a.N) continue;
                     if (a.epi == LIN_F32) {
                         float *y = (float *)a.y + (size_t)(row0 + c * CW) * a.N + n;
 #pragma unroll
@@ -237,17 +238,20 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                         }
                     }
                 } else {
+                    // lane j holds the pair (and its weight) of the block's token j
+                    const int my_row = row0 + c * CW + lane;
+                    const int my_pair = lane < CW && c * CW + lane < cnt ? a.r.perm[my_row] : 0;
+                    const float my_score = DUAL ? a.r.score[my_pair] : 0.f;
 #pragma unroll
                     for (int j = 0; j < CW; ++j) {
-                        if (c * CW + j >= cnt) break;
-                        const int row = row0 + c * CW + j, pair = a.r.perm[row];
-                        if (DUAL) {
-                            const float s = a.r.score[pair];
-                            ((__nv_bfloat16 *)a.y)[(size_t)row * a.N + n] = __float2bfloat16_rn(
-                                clamped_glu_value(s * __uint_as_float(v[j]), s * __uint_as_float(v[16 + j % 16]), a.limit));
-                        } else {
+                        const int pair = __shfl_sync(0xffffffffu, my_pair, j);
+                        const float sc = __shfl_sync(0xffffffffu, my_score, j);
+                        if (c * CW + j >= cnt || n >= a.N) continue;
+                        if (DUAL)
+                            ((__nv_bfloat16 *)a.y)[(size_t)(row0 + c * CW + j) * a.N + n] = __float2bfloat16_rn(
+                                clamped_glu_value(sc * __uint_as_float(v[j]), sc * __uint_as_float(v[16 + j % 16]), a.limit));
+                        else
                             ((float *)a.y)[(size_t)pair * a.N + n] = __uint_as_float(v[j]);
-                        }
                     }
                 }
             }
@@ -298,19 +302,24 @@ int launch_tc(const LinArgs &a, cudaStream_t s) {
 }  // namespace
 
 int gemm_bf16_tc(const LinArgs &a, int mode, cudaStream_t s) {
+    // The token tile: waves of tiles over the SMs times what a tile costs (its tokens, and a fixed part
+    // for the weight tile it streams and the hand-overs).  An expert's rows are counted with what
+    // routing spreads around their mean.
     const int sms = device_sm_count(), n_tiles = (a.N + 127) / 128;
-    auto tiles = [&](int ntok) { return (long long)n_tiles * ((a.M + ntok - 1) / ntok); };
+    const int groups = mode == LIN_DENSE ? 1 : std::min(a.r.E, a.r.pairs);
+    const double rows = mode == LIN_DENSE ? a.M : (double)a.M / groups + std::sqrt((double)a.M / groups);
+    auto cost = [&](int ntok) {
+        const double tiles = std::ceil(rows / ntok) * n_tiles * groups;
+        return std::ceil(tiles / sms) * (ntok + 40);
+    };
     if (mode == LIN_DENSE) {
-        // the widest token tile that still gives every SM one
-        if (tiles(256) >= sms) return launch_tc<256, LIN_DENSE>(a, s);
-        if (tiles(128) >= sms || a.M > 512) return launch_tc<128, LIN_DENSE>(a, s);
-        return launch_tc<64, LIN_DENSE>(a, s);
+        if (cost(256) <= cost(128) && cost(256) <= cost(64)) return launch_tc<256, LIN_DENSE>(a, s);
+        return cost(128) <= cost(64) ? launch_tc<128, LIN_DENSE>(a, s) : launch_tc<64, LIN_DENSE>(a, s);
     }
     AB2_REQUIRE(a.r.E <= GB_MAX_EXPERTS, AB2_ERR_UNSUPPORTED, "%d experts exceed the %d the grouped GEMM serves", a.r.E, GB_MAX_EXPERTS);
-    const int per_expert = (a.r.pairs + a.r.E - 1) / a.r.E;
-    if (mode == LIN_MOE_GLU) return per_expert > 96 ? launch_tc<128, LIN_MOE_GLU>(a, s) : launch_tc<64, LIN_MOE_GLU>(a, s);
-    if (per_expert > 192) return launch_tc<256, LIN_MOE_DOWN>(a, s);
-    return per_expert > 96 ? launch_tc<128, LIN_MOE_DOWN>(a, s) : launch_tc<64, LIN_MOE_DOWN>(a, s);
+    if (mode == LIN_MOE_GLU) return cost(128) <= cost(64) ? launch_tc<128, LIN_MOE_GLU>(a, s) : launch_tc<64, LIN_MOE_GLU>(a, s);
+    if (cost(256) <= cost(128) && cost(256) <= cost(64)) return launch_tc<256, LIN_MOE_DOWN>(a, s);
+    return cost(128) <= cost(64) ? launch_tc<128, LIN_MOE_DOWN>(a, s) : launch_tc<64, LIN_MOE_DOWN>(a, s);
 }
 
 }  // namespace ab2

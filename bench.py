@@ -357,8 +357,153 @@ def prefill_rows(torch, model, cache, prompt, B):
     return logits
 
 
+# Tovelix at layer sizes of real models, random weights.  "dense" is the closest existing decoder at
+# equal width, depth, heads and active feed-forward width: the dense GQA decoder, W4A16 g128, INT8 KV.
+TOVELIX = {
+    "w2048": dict(width=2048, layers="LLLALLLA", heads=16, kv_heads=4, window=1024, experts=32, top=4, ff=1024),
+    "w4096": dict(width=4096, layers="LLLALLLA", heads=32, kv_heads=8, window=2048, experts=8, top=2, ff=7168),
+}
+
+
+def build_tovelix(pkg, torch, c, max_tokens, max_seq, vocab=32000):
+    gen = torch.Generator(device="cuda").manual_seed(0)
+
+    def lin(n, k):
+        w = torch.empty((n, k), dtype=torch.bfloat16, device="cuda").normal_(generator=gen)
+        return pkg.QuantLinear.from_bf16(w.mul_(k ** -0.5))
+
+    d, H, G, E, ff = c["width"], c["heads"], c["kv_heads"], c["experts"], c["ff"]
+    ones = torch.ones(max(d, H * 128), device="cuda")
+    ffn = pkg.MoeFfn(E, c["top"], ff, 7.0)
+    weights = {"embedding": lin(vocab, d), "embed_norm": ones[:d], "final_norm": ones[:d]}
+    layers = []
+    for i, kind in enumerate(c["layers"]):
+        q = f"layers.{i}."
+        if kind == "L":
+            layers.append((pkg.LightningMixer(H, 128, 128, tuple(1 - 2.0 ** (-2 - 6 * h / H) for h in range(H))), ffn))
+            weights[q + "in"] = lin(4 * H * 128, d)
+            weights[q + "mix_norm"] = ones[:H * 128]
+        else:
+            layers.append((pkg.AttentionMixer(H, G, 128, 128, 0.0884, c["window"], 64, 10000.0, True, True, 0.5), ffn))
+            weights[q + "in"] = lin((H + 2 * G) * 128, d)
+        weights[q + "out"] = lin(d, H * 128)
+        weights[q + "norm1"] = weights[q + "norm2"] = ones[:d]
+        weights[q + "router"] = lin(E, d)
+        weights[q + "gate"], weights[q + "up"], weights[q + "down"] = lin(E * ff, d), lin(E * ff, d), lin(E * d, ff)
+    cfg = pkg.StackConfig(d, vocab, layers, max_seq)
+    return pkg.StackModel(cfg, weights, torch.bfloat16, max_tokens)
+
+
+def tovelix_step_bytes(c, batch, ctx, vocab=32000):
+    """Algorithmic bytes of a decode step: every weight a token uses once (experts: as many as the batch
+    can reach), the cached window, the states read and written."""
+    d, H, G = c["width"], c["heads"], c["kv_heads"]
+    hit = c["experts"] * (1 - (1 - c["top"] / c["experts"]) ** batch)
+    ffn = 2 * (c["experts"] * d + 3 * hit * d * c["ff"])
+    light = 2 * (5 * H * 128 * d) + batch * 2 * 4 * H * 128 * 128
+    attn = 2 * ((2 * H + 2 * G) * 128 * d) + batch * min(ctx, c["window"]) * 2 * 2 * G * 128
+    return sum(ffn + (light if k == "L" else attn) for k in c["layers"]) + 2 * vocab * d
+
+
+def tovelix_prefill_flops(c, S, vocab=32000):
+    d, H, G, W = c["width"], c["heads"], c["kv_heads"], c["window"]
+    ffn = 2 * S * d * (c["experts"] + 3 * c["top"] * c["ff"])
+    light = 2 * S * 5 * H * 128 * d + S * H * 4 * 128 * 128
+    keys = sum(min(i + 1, W) for i in range(S))
+    attn = 2 * S * (2 * H + 2 * G) * 128 * d + 4 * H * 128 * keys
+    return sum(ffn + (light if k == "L" else attn) for k in c["layers"]) + 2 * vocab * d
+
+
+def time_model(pkg, torch, model, vocab, kv_dtype, batches, prompts, steps, ctx=PROMPT):
+    """Decode ms per step at the given batches (context `ctx`) and prefill ms of the given prompt lengths."""
+    stream = torch.cuda.Stream()
+    out = {"decode": {}, "prefill": {}}
+    with torch.cuda.stream(stream):
+        for B in batches:
+            cache = model.empty_kv_cache_with_capacity(ctx + 5 * steps + 16, batch=B, dtype=kv_dtype)
+            # rows of one batch see different tokens, so that experts are shared as in serving
+            prompt = torch.randint(0, vocab, (B, ctx), generator=torch.Generator().manual_seed(3))
+            logits = torch.cat([model.forward_with_cache(prompt[b:b + 1], 0, cache, row=b, last_only=True).view(1, -1) for b in range(B)])
+            start, step, time_block, _ = decode_timer(torch, model, cache, pkg, B, stream, None, 1)
+            start(pkg.dispatch.argmax(logits))
+            for _ in range(4):
+                step()
+            blocks = sorted(time_block(steps) / steps for _ in range(3))
+            out["decode"][B] = blocks[1]
+            del cache
+        for S in prompts:
+            cache = model.empty_kv_cache_with_capacity(S + 8, batch=1, dtype=kv_dtype)
+            prompt = torch.randint(0, vocab, (1, S), generator=torch.Generator().manual_seed(2))
+            times = []
+            for i in range(7):
+                cache.truncate(0, 0)
+                stream.synchronize()
+                a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                a.record(stream)
+                model.forward_with_cache(prompt, 0, cache, row=0, last_only=True)
+                b.record(stream)
+                stream.synchronize()
+                times.append(a.elapsed_time(b))
+            out["prefill"][S] = sorted(times[2:])[2]
+            del cache
+    return out
+
+
+def tovelix_record(args):
+    """`--model tovelix`: decode and prefill throughput of the Tovelix stack beside the dense decoder of
+    equal width, depth, heads and active feed-forward width."""
+    import torch
+    torch.cuda.set_device(0)
+    from __graft_entry__ import import_package
+    pkg = import_package()
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    batches, prompts, vocab = (1, 8, 32), (512, 2048, 8192), 32000
+    sizes = {}
+    clocks = ClockSampler(0)
+    for name, c in TOVELIX.items():
+        if args.size not in ("all", name):
+            continue
+        model = build_tovelix(pkg, torch, c, max(prompts), max(prompts) + 512, vocab)
+        with clocks:
+            t = time_model(pkg, torch, model, vocab, "bf16", batches, prompts, args.steps)
+        del model
+        torch.cuda.empty_cache()
+        n = len(c["layers"])
+        dc = dict(n_layers=n, d_model=c["width"], n_heads=c["heads"], n_kv_heads=c["kv_heads"], head_dim=128,
+                  ffn_hidden=c["top"] * c["ff"], vocab=vocab, max_seq=max(prompts) + 512)
+        mc, weights = build_large(pkg, torch, dc)
+        dense = pkg.AarambhModel(mc, weights, dtype=torch.bfloat16, max_tokens=max(prompts))
+        with clocks:
+            u = time_model(pkg, torch, dense, vocab, "int8", batches, prompts, args.steps)
+        del dense, weights
+        torch.cuda.empty_cache()
+        rec = {"config": dict(c, vocab=vocab, head_dim=128), "decode": {}, "prefill": {}}
+        for B in batches:
+            byt, dbyt = tovelix_step_bytes(c, B, PROMPT), step_weight_bytes(dc) + B * PROMPT * kv_bytes_per_token(dc)
+            rec["decode"][f"batch{B}"] = {
+                "ms": round(t["decode"][B], 4), "tok_s": round(B * 1e3 / t["decode"][B], 1), "hbm_frac": round(byt / t["decode"][B] / 1e6 / hbm, 4),
+                "dense_w4a16": {"ms": round(u["decode"][B], 4), "tok_s": round(B * 1e3 / u["decode"][B], 1),
+                                "hbm_frac": round(dbyt / u["decode"][B] / 1e6 / hbm, 4)}}
+        for S in prompts:
+            fl = tovelix_prefill_flops(c, S)
+            dfl = 2.0 * S * sum(a * b for a, b in linear_shapes(dc).values()) * n + 2.0 * vocab * c["width"] + n * 2.0 * c["heads"] * 128 * S * (S + 1)
+            rec["prefill"][f"{S}"] = {
+                "ms": round(t["prefill"][S], 3), "tok_s": round(S * 1e3 / t["prefill"][S], 1), "bf16_frac": round(fl / t["prefill"][S] / 1e9 / tf, 4),
+                "dense_w4a16": {"ms": round(u["prefill"][S], 3), "tok_s": round(S * 1e3 / u["prefill"][S], 1),
+                                "bf16_frac": round(dfl / u["prefill"][S] / 1e9 / tf, 4)}}
+        sizes[name] = rec
+    first = next(iter(sizes.values()))["decode"]["batch1"]
+    return {"metric": "Tovelix decode tok/s", "value": first["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": 4,
+            "ms_per_step": first["ms"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"workload": "tovelix", "context": PROMPT, "l2": "the weights of a step exceed the 126 MB L2"},
+            "sizes": sizes, "clocks": clocks.summary(), "device_status": pkg.device_status()}
+
+
 def main():
     ap = argparse.ArgumentParser()
+    ap.add_argument("--model", default="dense", choices=["dense", "tovelix"], help="dense: the default workload")
+    ap.add_argument("--size", default="all", choices=["all"] + list(TOVELIX), help="tovelix: one size only")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
@@ -376,6 +521,11 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     cfg = LARGE
     B = args.batch
+
+    if args.model == "tovelix":
+        if rank == 0:
+            print(json.dumps(tovelix_record(args)))
+        return 0
 
     if args.cpu_ops:
         if rank == 0:

@@ -294,9 +294,95 @@ def bench_step(pkg, args):
                       "us_per_step": round(a.elapsed_time(b) * 1e3 / 32, 2)}), flush=True)
 
 
+def report(kernel, t, byt=None, flops=None, **what):
+    rec = dict(kernel=kernel, **what, us=round(t * 1e6, 2))
+    if byt:
+        rec.update(GBs=round(byt / t / 1e9, 1), frac_of_measured_hbm=round(byt / t / 1e9 / peak_hbm(), 3))
+    if flops:
+        rec.update(TFLOPs=round(flops / t / 1e12, 1), frac_of_measured_bf16=round(flops / t / 1e12 / peak_tflops(), 3))
+    print(json.dumps(rec), flush=True)
+
+
+def bench_stack(pkg, args):
+    """The kernels of layer stacks, each in a graph over operands that exceed L2 (several weights or caches
+    in turn): dense bf16 linears, mixture of experts, window attention, lightning attention."""
+    stream = torch.cuda.Stream()
+    only = args.only.split(",") if args.only else ["linear", "moe", "window", "lightning"]
+
+    def lin(n, k):
+        return pkg.QuantLinear.from_bf16(torch.empty((n, k), dtype=torch.bfloat16, device="cuda").normal_().mul_(k ** -0.5))
+
+    def x_of(*shape):
+        return torch.randn(*shape, device="cuda").to(torch.bfloat16)
+
+    if "linear" in only:
+        for K, N in SHAPES:
+            w = [lin(N, K) for _ in range(max(2, math.ceil(400e6 / (2 * K * N))))]
+            for M in (1, 8, 32, 512, 2048, 8192):
+                x = x_of(M, K)
+                t = time_graph(lambda: [l(x) for l in w], 5, stream) / len(w)
+                byt, fl = 2 * (K * N + M * (K + N)), 2.0 * M * K * N
+                if M <= 32:
+                    report("gemv_bf16_kernel", t, byt=byt, K=K, N=N, M=M)
+                else:
+                    report("gemm_bf16_tc_kernel", t, flops=fl, K=K, N=N, M=M)
+            del w
+    if "moe" in only:
+        for d, E, top, ff in ((2048, 32, 4, 1024), (4096, 8, 2, 7168)):
+            ffn = pkg.MoeFfn(E, top, ff, 7.0)
+            layers = [pkg.dispatch.MoeExperts(ffn, lin(E, d), lin(E * ff, d), lin(E * ff, d), lin(E * d, ff)) for _ in range(2)]
+            for T in (1, 8, 32, 512, 2048, 8192):
+                x, out = x_of(T, d), torch.empty((T, top, d), device="cuda")
+                t = time_graph(lambda: [l(x, out) for l in layers], 5, stream) / 2
+                hit = E * (1 - (1 - top / E) ** T)
+                if T <= 32:
+                    report("mixture of experts (route, gemv_bf16 x 3)", t, byt=2 * (E * d + 3 * hit * d * ff), width=d, E=E, top=top, ff=ff, T=T)
+                else:
+                    report("mixture of experts (route, gather, gemm_bf16_tc x 2)", t, flops=2.0 * T * top * 3 * d * ff, width=d, E=E, top=top, ff=ff, T=T)
+            del layers
+    H, G = 32, 8
+    if "window" in only:
+        for W, ctx, B in ((1024, 4096, 1), (1024, 4096, 32), (4096, 8192, 1), (4096, 8192, 32), (0, 32768, 8)):
+            cfg = pkg.StackConfig(64, 64, [(pkg.AttentionMixer(H, G, 128, 128, 0.09, W), None)], ctx)
+            caches = [pkg.KVCache.for_stack(cfg, ctx, B, 512, "bf16") for _ in range(max(1, min(8, int(400e6 / (B * min(W or ctx, ctx) * 4 * G * 128)))))]
+            for c in caches:
+                c.commit(ctx - 8, 0, B)
+            qkv = x_of(B, 1, (H + 2 * G) * 128)
+            t = time_graph(lambda: [pkg.dispatch.window_attention(c, cfg, 0, qkv, None, 1e-5) for c in caches], 5, stream) / len(caches)
+            report("window attention, decode", t, byt=B * min(W or ctx, ctx) * 4 * G * 128, window=W, ctx=ctx, B=B)
+            del caches
+        for W, S in ((1024, 512), (1024, 2048), (1024, 8192), (4096, 8192), (0, 2048)):
+            cfg = pkg.StackConfig(64, 64, [(pkg.AttentionMixer(H, G, 128, 128, 0.09, W), None)], S)
+            cache = pkg.KVCache.for_stack(cfg, S, 1, S, "bf16")
+            qkv = x_of(1, S, (H + 2 * G) * 128)
+            t = time_graph(lambda: pkg.dispatch.window_attention(cache, cfg, 0, qkv, None, 1e-5), 5, stream)
+            keys = sum(min(i + 1, W or S) for i in range(S))
+            report("window_attn_mma_kernel (and preparation)", t, flops=4.0 * H * 128 * keys, window=W, S=S)
+            del cache
+    if "lightning" in only:
+        decay = tuple(1 - 2.0 ** (-2 - 6 * h / H) for h in range(H))
+        powers = pkg.dispatch.decay_powers(decay)
+        cfg = pkg.StackConfig(64, 64, [(pkg.LightningMixer(H, 128, 128, decay), None)], 1 << 20)
+        for B in (1, 8, 32):
+            caches = [pkg.KVCache.for_stack(cfg, 1 << 20, B, 8192, "bf16") for _ in range(max(2, 400 // (2 * B)))]
+            for c in caches:
+                c.commit(4, 0, B)
+            qkv = x_of(B, 1, 4 * H * 128)
+            t = time_graph(lambda: [pkg.dispatch.lightning_attention(c, cfg, 0, qkv, powers) for c in caches], 5, stream) / len(caches)
+            report("lightning_serial_kernel, decode", t, byt=B * H * 128 * 128 * 8, B=B)
+            del caches
+        for B, S in ((1, 512), (1, 2048), (1, 8192), (4, 2048)):
+            cache = pkg.KVCache.for_stack(cfg, 1 << 20, B, 8192, "bf16")
+            qkv = x_of(B, S, 4 * H * 128)
+            t = time_graph(lambda: pkg.dispatch.lightning_attention(cache, cfg, 0, qkv, powers), 5, stream)
+            report("lightning_chunk_kernel", t, byt=B * S * H * 128 * (3 * 2 + 4), flops=B * S * H * 4.0 * 128 * 128, B=B, S=S)
+            del cache
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemv", "gemm", "attention", "prefill_attention", "step"])
+    ap.add_argument("what", choices=["gemv", "gemm", "attention", "prefill_attention", "step", "stack"])
+    ap.add_argument("--only", default=None, help="stack: linear, moe, window, lightning")
     ap.add_argument("--layers", type=int, default=2)
     ap.add_argument("--ctx", type=int, default=512)
     ap.add_argument("--batch", type=int, default=1, help="step: sequences decoded together")
@@ -319,6 +405,8 @@ def main():
         bench_gemm(pkg, args)
     elif args.what == "step":
         bench_step(pkg, args)
+    elif args.what == "stack":
+        bench_stack(pkg, args)
     elif args.what == "prefill_attention":
         args.cases = [tuple(int(v) for v in c.split("x")) for c in (args.cases or "1x512,1x2048,4x512").split(",")]
         bench_prefill_attention(pkg, args)
