@@ -86,7 +86,7 @@ SIGNATURES = {
     "ab2_kv_clone": ([_pp, _p, _p], _i),
     "ab2_kv_read": ([_p, _i, _i, _p, _p, _p], _i),
     "ab2_window_attention": ([_p, _i, _p, _p, _p, _i, _p, _p, _f, _p, _i, _i, _i, _i, _p], _i),
-    "ab2_lightning_attention": ([_p, _i, _p, _p, _p, C.c_longlong, _p, _i, _i, _i, _i, _p], _i),
+    "ab2_lightning_attention": ([_p, _i, _p, _p, _p, C.c_longlong, _p, _p, _i, _i, _i, _i, _p], _i),
     "ab2_moe_workspace": ([_p, _i, _i, _i, C.POINTER(C.c_size_t)], _i),
     "ab2_moe_forward": ([_p, _p, _p, _p, _p, _p, _i, _i, _p, _p, _p], _i),
     "ab2_attention_decode": ([_p, _i, _p, _p, _i, _i, _f, _i, _p], _i),

@@ -7,6 +7,7 @@
 //   window_attn_kernel         f32 arithmetic on CUDA cores: decode (the window split over CTAs,
 //                              log-sum-exp merge), f32 models, unusual head sizes
 //   window_attn_mma_kernel     prompts in bf16 on the warp-level tensor cores
+//   window_decode_mma_kernel   decode in bf16, preparation included, on the warp-level tensor cores
 //
 // Scores, softmax weights and sums are f32 throughout.  The tensor-core kernel multiplies the
 // weights with the values as two bf16 terms (the rounded weight and what rounding left), so the
@@ -23,6 +24,34 @@ int device_sm_count();
 namespace {
 
 constexpr int MAX_DIM = 256;
+
+// Rotation and normalisation of one head by one warp: lane j holds the pairs j, j + 32, ... of `src`
+// (NP of them at most) in u and w.
+template <typename T, int NP>
+__device__ __forceinline__ void rotate_normalise(const WindowPrepArgs &a, const T *src, int pos, int lane, float (&u)[NP], float (&w)[NP]) {
+    const int half = (a.dim + 1) >> 1;
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+        const int i = lane + 32 * j;
+        u[j] = w[j] = 0.f;
+        if (i >= half) continue;
+        float x0 = to_f32(src[2 * i]), x1 = 2 * i + 1 < a.dim ? to_f32(src[2 * i + 1]) : 0.f;
+        if (2 * i < a.rot_dims) {
+            const size_t t = (size_t)pos * (a.rot_dims >> 1) + i;
+            const float c = a.cos_t[t], sn = a.sin_t[t], r0 = x0 * c - x1 * sn, r1 = x1 * c + x0 * sn;
+            x0 = r0; x1 = r1;
+        }
+        u[j] = x0; w[j] = x1;
+        sum = fmaf(x0, x0, fmaf(x1, x1, sum));
+    }
+    if (!a.qk_norm) return;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    const float inv = 1.f / sqrtf(sum / (float)a.dim + a.eps);
+#pragma unroll
+    for (int j = 0; j < NP; ++j) { u[j] *= inv; w[j] *= inv; }
+}
 
 // One warp per (token, head): H query heads, then G key heads, then G value heads.
 template <typename T>
@@ -51,34 +80,15 @@ __global__ void __launch_bounds__(256) window_prep_kernel(WindowPrepArgs a) {
     }
     src += (size_t)vec * a.dim;
     const int half = (a.dim + 1) >> 1;
-    float u[MAX_DIM / 64], w[MAX_DIM / 64], sum = 0.f;
-#pragma unroll
-    for (int j = 0; j < MAX_DIM / 64; ++j) {
-        const int i = lane + 32 * j;
-        u[j] = w[j] = 0.f;
-        if (i >= half) continue;
-        float x0 = to_f32(src[2 * i]), x1 = 2 * i + 1 < a.dim ? to_f32(src[2 * i + 1]) : 0.f;
-        if (2 * i < a.rot_dims) {
-            const size_t t = (size_t)pos * (a.rot_dims >> 1) + i;
-            const float c = a.cos_t[t], sn = a.sin_t[t], r0 = x0 * c - x1 * sn, r1 = x1 * c + x0 * sn;
-            x0 = r0; x1 = r1;
-        }
-        u[j] = x0; w[j] = x1;
-        sum = fmaf(x0, x0, fmaf(x1, x1, sum));
-    }
-    float inv = 1.f;
-    if (a.qk_norm) {
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        inv = 1.f / sqrtf(sum / (float)a.dim + a.eps);
-    }
+    float u[MAX_DIM / 64], w[MAX_DIM / 64];
+    rotate_normalise<T, MAX_DIM / 64>(a, src, pos, lane, u, w);
     T *dst = vec < a.H ? src : (T *)l.k + (((size_t)row * a.G + (vec - a.H)) * l.cap + slot) * l.kds;
 #pragma unroll
     for (int j = 0; j < MAX_DIM / 64; ++j) {
         const int i = lane + 32 * j;
         if (i >= half) continue;
-        dst[2 * i] = from_f32<T>(u[j] * inv);
-        if (2 * i + 1 < a.dim) dst[2 * i + 1] = from_f32<T>(w[j] * inv);
+        dst[2 * i] = from_f32<T>(u[j]);
+        if (2 * i + 1 < a.dim) dst[2 * i + 1] = from_f32<T>(w[j]);
     }
 }
 
@@ -415,11 +425,14 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
 }
 
 // ---------------------------------------------------------------------------
-// Decode in bf16: one query per sequence.  The (up to 16) query heads of a KV head are the rows of
-// the MMA, the keys its columns.  grid (nsplit, G * head groups, rows), 4 warps: a CTA takes one of
-// nsplit runs of the visible keys and its warps deal them out 16 at a time; a warp streams its keys and
-// values through a ring of its own in shared memory (cp.async, no CTA barrier in the loop).  The warps
-// meet in shared memory at the end, the splits in window_merge_kernel.
+// Decode in bf16: one query per sequence, one launch.  The (up to 16) query heads of a KV head are the
+// rows of the MMA, the keys its columns.  grid (nsplit, G * head groups, rows), 4 warps.
+//   - The cached keys of the window are cut into nsplit runs; a CTA's warps deal its run out 16 at a time
+//     and stream it through rings of their own in shared memory (cp.async, no CTA barrier in the loop).
+//     The first of it is requested before the dependency wait: it belongs to earlier steps.
+//   - Every CTA rotates and normalises its query heads; the last split also the new key, mixes the new
+//     value, stores both in the cache and attends to them from shared memory.
+//   - The warps meet in shared memory, the splits in the CTA that arrives last.
 // ---------------------------------------------------------------------------
 constexpr int WD_STAGES = 3;
 
@@ -427,20 +440,22 @@ template <int DP, int VP>
 __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int KB = 16 * DP * 2, VB = 16 * VP * 2, STAGE = KB + VB;
+    __shared__ __align__(128) uint8_t fresh[STAGE];            // the new token's key and value as row 0 of a tile
+    __shared__ __align__(16) __nv_bfloat16 qs[16][DP + 8];
     __shared__ float wm[4][16], wl[4][16];
-    pdl_wait();
-    pdl_launch_dependents();
     const KvLayer &l = a.kv.l;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
     const int groups = (a.rep + 15) / 16, kvh = blockIdx.y / groups, hg = blockIdx.y % groups;
     const int head0 = kvh * a.rep + hg * 16, nh = min(16, a.rep - hg * 16);
     const int rrow = blockIdx.z, row = kv_row(a.kv, a.row0, rrow);
-    const int pos = a.kv.lens[row], lo = max(0, pos - l.window + 1), n = pos + 1 - lo;
+    const int pos = a.kv.lens[row], lo = max(0, pos - l.window + 1), n = pos - lo;  // cached keys in sight
     const int per = ((n + a.nsplit - 1) / a.nsplit + 63) & ~63;
-    const int j0 = lo + (int)blockIdx.x * per, j1 = min(pos + 1, j0 + per);
-    const __nv_bfloat16 *kb = (const __nv_bfloat16 *)l.k + ((size_t)row * l.kvh + kvh) * l.cap * l.kds;
-    const __nv_bfloat16 *vb = (const __nv_bfloat16 *)l.v + ((size_t)row * l.kvh + kvh) * l.cap * l.vds;
+    const int j0 = lo + (int)blockIdx.x * per, j1 = min(pos, j0 + per);
+    const bool owns_new = (int)blockIdx.x == a.nsplit - 1;
+    __nv_bfloat16 *kb = (__nv_bfloat16 *)l.k + ((size_t)row * l.kvh + kvh) * l.cap * l.kds;
+    __nv_bfloat16 *vb = (__nv_bfloat16 *)l.v + ((size_t)row * l.kvh + kvh) * l.cap * l.vds;
     const uint32_t ring = (uint32_t)__cvta_generic_to_shared(smem) + warp * WD_STAGES * STAGE;
+    const uint32_t fresh_s = (uint32_t)__cvta_generic_to_shared(fresh);
 
     auto load = [&](int base, int st) {
         if (base < j1) {
@@ -467,21 +482,58 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
     };
 #pragma unroll
     for (int st = 0; st < WD_STAGES - 1; ++st) load(j0 + (st * 4 + warp) * 16, st);
+    for (int i = threadIdx.x; i < STAGE / 16; i += 128) reinterpret_cast<uint4 *>(fresh)[i] = make_uint4(0u, 0u, 0u, 0u);
+    for (int i = threadIdx.x; i < 16 * (DP + 8) / 8; i += 128) reinterpret_cast<uint4 *>(&qs[0][0])[i] = make_uint4(0u, 0u, 0u, 0u);
+    __syncthreads();
+    pdl_wait();
+    pdl_launch_dependents();
+
+    {
+        const WindowPrepArgs &p = a.prep;
+        const __nv_bfloat16 *tok = (const __nv_bfloat16 *)p.qkv + (size_t)rrow * p.stride;
+        constexpr int NP = DP / 64;
+        float u[NP], w[NP];
+        for (int h = warp; h < nh; h += 4) {
+            rotate_normalise<__nv_bfloat16, NP>(p, tok + (size_t)(head0 + h) * p.dim, pos, lane, u, w);
+#pragma unroll
+            for (int j = 0; j < NP; ++j)
+                if (2 * (lane + 32 * j) < p.dim)
+                    *reinterpret_cast<__nv_bfloat162 *>(&qs[h][2 * (lane + 32 * j)]) = __floats2bfloat162_rn(u[j], w[j]);
+        }
+        const int slot = pos % l.cap;
+        if (owns_new && warp == 3) {
+            rotate_normalise<__nv_bfloat16, NP>(p, tok + (size_t)(p.H + kvh) * p.dim, pos, lane, u, w);
+#pragma unroll
+            for (int j = 0; j < NP; ++j) {
+                const int d = 2 * (lane + 32 * j);
+                if (d >= p.dim) continue;
+                const __nv_bfloat162 kv2 = __floats2bfloat162_rn(u[j], w[j]);
+                *reinterpret_cast<__nv_bfloat162 *>(fresh + d * 2) = kv2;  // row 0: chunk order is the plain one
+                if (hg == 0) *reinterpret_cast<__nv_bfloat162 *>(kb + (size_t)slot * l.kds + d) = kv2;
+            }
+        }
+        if (owns_new && warp == 2) {
+            const __nv_bfloat16 *src = tok + (size_t)(p.H + p.G) * p.dim + (size_t)kvh * p.vdim;
+            __nv_bfloat16 *first = (__nv_bfloat16 *)p.v_first + ((size_t)rrow * p.G + kvh) * p.vdim;
+            for (int d = lane; d < p.vdim; d += 32) {
+                __nv_bfloat16 v = src[d];
+                if (p.v_mode == 1 && hg == 0) first[d] = v;
+                if (p.v_mode == 2) v = __float2bfloat16_rn((1.f - p.lambda) * __bfloat162float(v) + p.lambda * __bfloat162float(first[d]));
+                *reinterpret_cast<__nv_bfloat16 *>(fresh + KB + d * 2) = v;
+                if (hg == 0) vb[(size_t)slot * l.vds + d] = v;
+            }
+        }
+    }
+    __syncthreads();
 
     uint32_t qf[DP / 16][4];
-    {
-        const __nv_bfloat16 *ra = (const __nv_bfloat16 *)a.q + (size_t)rrow * a.q_stride + (size_t)(head0 + min(g, nh - 1)) * a.dim;
-        const __nv_bfloat16 *rb = (const __nv_bfloat16 *)a.q + (size_t)rrow * a.q_stride + (size_t)(head0 + min(g + 8, nh - 1)) * a.dim;
 #pragma unroll
-        for (int ks = 0; ks < DP / 16; ++ks)
+    for (int ks = 0; ks < DP / 16; ++ks)
 #pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int d = ks * 16 + h * 8 + 2 * c;
-                const bool in = d < a.dim;
-                qf[ks][2 * h] = in ? *reinterpret_cast<const uint32_t *>(ra + d) : 0u;
-                qf[ks][2 * h + 1] = in ? *reinterpret_cast<const uint32_t *>(rb + d) : 0u;
-            }
-    }
+        for (int h = 0; h < 2; ++h) {
+            qf[ks][2 * h] = *reinterpret_cast<const uint32_t *>(&qs[g][ks * 16 + h * 8 + 2 * c]);
+            qf[ks][2 * h + 1] = *reinterpret_cast<const uint32_t *>(&qs[g + 8][ks * 16 + h * 8 + 2 * c]);
+        }
     const float sl = a.scale * 1.44269504088896341f;  // scores in powers of two
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f}, o[VP / 8][4];
 #pragma unroll
@@ -489,12 +541,9 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
 
-    int st = 0;
-    for (int base = j0 + warp * 16; base < j1; base += 64) {
-        load(base + (WD_STAGES - 1) * 64, (st + WD_STAGES - 1) % WD_STAGES);
-        asm volatile("cp.async.wait_group %0;\n" ::"n"(WD_STAGES - 1) : "memory");
-        __syncwarp();
-        const uint32_t ks0 = ring + st * STAGE, vs0 = ks0 + KB;
+    // 16 keys in shared memory, the first `live` of which count
+    auto attend = [&](uint32_t ks0, int live) {
+        const uint32_t vs0 = ks0 + KB;
         float s[2][4], bm[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
@@ -512,13 +561,13 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
             }
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                s[nt][j] = base + nt * 8 + 2 * c + (j & 1) < j1 ? s[nt][j] * sl : -INFINITY;
+                s[nt][j] = nt * 8 + 2 * c + (j & 1) < live ? s[nt][j] * sl : -INFINITY;
                 bm[j >> 1] = fmaxf(bm[j >> 1], s[nt][j]);
             }
         }
         float corr[2];
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {  // every 16 keys hold at least one of the run: the maximum is finite
+        for (int h = 0; h < 2; ++h) {  // live > 0: the maximum is finite
             bm[h] = fmaxf(bm[h], __shfl_xor_sync(0xffffffffu, bm[h], 1));
             bm[h] = fmaxf(bm[h], __shfl_xor_sync(0xffffffffu, bm[h], 2));
             const float m_new = fmaxf(m_run[h], bm[h]);
@@ -552,11 +601,20 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
             mma_bf16(o[2 * vv + 1], hi, b2, b3);
             mma_bf16(o[2 * vv + 1], lw, b2, b3);
         }
-        // The products above have consumed every matrix load of this stage (a tensor-core instruction
-        // waits for its operands), so the refill two statements into the next pass cannot overtake them.
+    };
+
+    int st = 0;
+    for (int base = j0 + warp * 16; base < j1; base += 64) {
+        load(base + (WD_STAGES - 1) * 64, (st + WD_STAGES - 1) % WD_STAGES);
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(WD_STAGES - 1) : "memory");
+        __syncwarp();
+        attend(ring + st * STAGE, j1 - base);
+        // The products have consumed every matrix load of this stage (a tensor-core instruction waits for
+        // its operands), so the refill at the top of the next pass cannot overtake them.
         __syncwarp();
         st = (st + 1) % WD_STAGES;
     }
+    if (owns_new && warp == 0) attend(fresh_s, 1);
     asm volatile("cp.async.wait_group 0;\n" ::: "memory");
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -571,6 +629,8 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
 #pragma unroll
         for (int j = 0; j < 4; ++j) wacc[((size_t)warp * 16 + g + 8 * (j >> 1)) * VP + i * 8 + 2 * c + (j & 1)] = o[i][j];
     __syncthreads();
+    __nv_bfloat16 *out = (__nv_bfloat16 *)a.out + ((size_t)rrow * a.H + head0) * a.vdim;
+    const size_t p0 = ((size_t)rrow * a.H + head0) * a.nsplit;
     for (int i = threadIdx.x; i < nh * a.vdim; i += 128) {
         const int hh = i / a.vdim, d = i % a.vdim;
         const float M = fmaxf(fmaxf(wm[0][hh], wm[1][hh]), fmaxf(wm[2][hh], wm[3][hh]));
@@ -581,15 +641,60 @@ __global__ void __launch_bounds__(128) window_decode_mma_kernel(WindowAttnArgs a
             L += e * wl[w][hh];
             A += e * wacc[((size_t)w * 16 + hh) * VP + d];
         }
-        const int head = head0 + hh;
         if (a.nsplit == 1) {
-            ((__nv_bfloat16 *)a.out)[((size_t)rrow * a.H + head) * a.vdim + d] = __float2bfloat16_rn(A / L);
+            out[i] = __float2bfloat16_rn(A / L);
         } else {
-            const size_t pi = ((size_t)rrow * a.H + head) * a.nsplit + blockIdx.x;
+            const size_t pi = p0 + (size_t)hh * a.nsplit + blockIdx.x;
             a.part_acc[pi * a.vdim + d] = A;
-            // the merge works in natural exponents
-            if (d == 0) { a.part_ml[pi * 2] = M * 0.693147180559945309f; a.part_ml[pi * 2 + 1] = L; }
+            if (d == 0) { a.part_ml[pi * 2] = M; a.part_ml[pi * 2 + 1] = L; }
         }
+    }
+    if (a.nsplit == 1) return;
+    // the CTA that arrives last merges the splits
+    __shared__ int last;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int *counter = a.counters + (size_t)rrow * gridDim.y + blockIdx.y;
+        last = atomicAdd(counter, 1) == a.nsplit - 1;
+        if (last) *counter = 0;  // at rest for the next launch
+    }
+    __syncthreads();
+    if (!last) return;
+    __threadfence();
+    // split weights per head, normalised, in shared memory ([nh][nsplit] floats; nsplit <= 64)
+    float *wt = reinterpret_cast<float *>(smem);
+    for (int hh = warp; hh < nh; hh += 4) {
+        const float *ml = a.part_ml + (p0 + (size_t)hh * a.nsplit) * 2;
+        float m[2], ls[2], M = -INFINITY, L = 0.f;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int sp = lane + 32 * k;
+            m[k] = sp < a.nsplit ? __ldcg(ml + sp * 2) : -INFINITY;
+            ls[k] = sp < a.nsplit ? __ldcg(ml + sp * 2 + 1) : 0.f;
+            M = fmaxf(M, m[k]);
+        }
+#pragma unroll
+        for (int q = 16; q > 0; q >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, q));
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            m[k] = m[k] == -INFINITY ? 0.f : exp2f(m[k] - M);
+            L = fmaf(m[k], ls[k], L);
+        }
+#pragma unroll
+        for (int q = 16; q > 0; q >>= 1) L += __shfl_xor_sync(0xffffffffu, L, q);
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (lane + 32 * k < a.nsplit) wt[hh * a.nsplit + lane + 32 * k] = m[k] / L;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < nh * a.vdim; i += 128) {
+        const int hh = i / a.vdim, d = i % a.vdim;
+        const float *acc = a.part_acc + (p0 + (size_t)hh * a.nsplit) * a.vdim + d;
+        float A = 0.f;
+#pragma unroll 8
+        for (int k = 0; k < a.nsplit; ++k) A = fmaf(wt[hh * a.nsplit + k], __ldcg(acc + (size_t)k * a.vdim), A);
+        out[i] = __float2bfloat16_rn(A);
     }
 }
 
@@ -634,6 +739,11 @@ int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cu
     cudaError_t e;
     const KvLayer &l = a.kv.l;
     const bool on_mma = sizeof(T) == 2 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 128 && a.vdim <= 128 && a.q_stride % 2 == 0;
+    if (!(on_mma && a.S == 1)) {
+        const dim3 pgrid((a.H + 2 * a.prep.G + 7) / 8, a.S, nrows);
+        e = launch_kernel(window_prep_kernel<T>, pgrid, dim3(256), 0, s, a.prep);
+        if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window preparation launch failed: %s", cudaGetErrorString(e));
+    }
     if (on_mma && a.S >= 16) {
         if (a.dim <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, nrows, s) : launch_mma<64, 128>(a, nrows, s);
         else e = a.vdim <= 64 ? launch_mma<128, 64>(a, nrows, s) : launch_mma<128, 128>(a, nrows, s);
@@ -648,8 +758,6 @@ int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cu
         const dim3 grid(a.nsplit, l.kvh * ((a.rep + 15) / 16), nrows);
         if (a.dim <= 64) e = a.vdim <= 64 ? launch_decode<64, 64>(a, grid, s) : launch_decode<64, 128>(a, grid, s);
         else e = a.vdim <= 64 ? launch_decode<128, 64>(a, grid, s) : launch_decode<128, 128>(a, grid, s);
-        if (e == cudaSuccess && a.nsplit > 1)
-            e = launch_kernel(window_merge_kernel<T>, dim3(a.H, nrows), dim3(std::min(128, (a.vdim + 31) / 32 * 32)), 0, s, a);
         if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window attention launch failed: %s", cudaGetErrorString(e));
         return AB2_OK;
     }
@@ -674,16 +782,8 @@ int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cu
 
 }  // namespace
 
-int window_prep(const WindowPrepArgs &a, int nrows, ab2_dtype dtype, cudaStream_t s) {
-    const dim3 grid((a.H + 2 * a.G + 7) / 8, a.S, nrows);
-    cudaError_t e = dtype == AB2_F32 ? launch_kernel(window_prep_kernel<float>, grid, dim3(256), 0, s, a)
-                                     : launch_kernel(window_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a);
-    if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window preparation launch failed: %s", cudaGetErrorString(e));
-    return AB2_OK;
-}
-
 int window_attention(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, ab2_dtype dtype, cudaStream_t s) {
-    a.part_acc = kv->part_acc; a.part_ml = kv->part_ml;
+    a.part_acc = kv->part_acc; a.part_ml = kv->part_ml; a.counters = kv->counters;
     return dtype == AB2_F32 ? launch_window<float>(kv, a, nrows, max_len, s) : launch_window<__nv_bfloat16>(kv, a, nrows, max_len, s);
 }
 

@@ -302,15 +302,15 @@ int launch_tc(const LinArgs &a, cudaStream_t s) {
 }  // namespace
 
 int gemm_bf16_tc(const LinArgs &a, int mode, cudaStream_t s) {
-    // The token tile: waves of tiles over the SMs times what a tile costs (its tokens, and a fixed part
-    // for the weight tile it streams and the hand-overs).  An expert's rows are counted with what
+    // The token tile: waves of tiles over the SMs times what a tile costs, which is the rows it streams
+    // through L2 - its tokens and the 128 (gate and up: 256) weight rows.  An expert's rows are counted with what
     // routing spreads around their mean.
     const int sms = device_sm_count(), n_tiles = (a.N + 127) / 128;
     const int groups = mode == LIN_DENSE ? 1 : std::min(a.r.E, a.r.pairs);
     const double rows = mode == LIN_DENSE ? a.M : (double)a.M / groups + std::sqrt((double)a.M / groups);
     auto cost = [&](int ntok) {
         const double tiles = std::ceil(rows / ntok) * n_tiles * groups;
-        return std::ceil(tiles / sms) * (ntok + 40);
+        return std::ceil(tiles / sms) * (ntok + (mode == LIN_MOE_GLU ? 256 : 128));
     };
     if (mode == LIN_DENSE) {
         if (cost(256) <= cost(128) && cost(256) <= cost(64)) return launch_tc<256, LIN_DENSE>(a, s);

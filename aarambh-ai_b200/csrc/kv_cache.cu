@@ -255,7 +255,7 @@ AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n
     for (int i = 0; i < batch; ++i) kv->saved_len[i] = -1;
     const int esz = (int)kv_elem_size(dtype);
     kv->max_splits = AB2_KV_MAX_SPLITS;
-    size_t part = 0, heads = 0;
+    size_t part = 0, heads = 0;  // an attention layer has at most `heads` (KV head, head group) pairs
     cudaError_t e = cudaSuccess;
     for (int i = 0; i < n_layers && e == cudaSuccess; ++i) {
         const ab2_layer_spec &sp = specs[i];
@@ -290,6 +290,9 @@ AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n
     kv->part_ml_bytes = (size_t)batch * kv->max_splits * heads * 2 * 4;
     if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_acc, kv->part_acc_bytes);
     if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_ml, kv->part_ml_bytes);
+    kv->counter_bytes = (size_t)batch * heads * 4;
+    if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->counters, kv->counter_bytes);
+    if (e == cudaSuccess && part > 0) e = cudaMemset(kv->counters, 0, kv->counter_bytes);
     if (e != cudaSuccess) {
         ab2_kv_destroy(kv);
         return fail(AB2_ERR_CUDA, "KV cache allocation failed: %s", cudaGetErrorString(e));
@@ -450,6 +453,7 @@ static int clone_stack(ab2_kv **out, const ab2_kv *src, cudaStream_t s) {
     for (int i = 0; i < src->B; ++i) { kv->high_host[i] = src->high_host[i]; kv->saved_len[i] = -1; }
     kv->lens_dev = kv->lens_host = kv->rows_dev = kv->rows_host = nullptr;
     kv->part_acc = kv->part_ml = nullptr;
+    kv->counters = nullptr;
     kv->rows_on = false;
     cudaError_t e = cudaSuccess;
     auto dup = [&](void **dst, const void *from, size_t bytes, bool contents) {
@@ -473,6 +477,7 @@ static int clone_stack(ab2_kv **out, const ab2_kv *src, cudaStream_t s) {
     dup((void **)&kv->rows_dev, src->rows_dev, (size_t)src->B * 4, false);
     dup((void **)&kv->part_acc, src->part_acc, src->part_acc_bytes, false);
     dup((void **)&kv->part_ml, src->part_ml, src->part_ml_bytes, false);
+    dup((void **)&kv->counters, src->counters, src->counter_bytes, true);  // at rest, as the source's
     if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->lens_host, (size_t)src->B * 4);
     if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->rows_host, (size_t)src->B * 4);
     if (e == cudaSuccess) e = cudaStreamSynchronize(s);

@@ -39,7 +39,7 @@ struct ab2_kv {
     KvLayer *layers;
     int *high_host;   // [B] most tokens a row has held since it was last empty (which ring slots are intact)
     int *saved_len;   // [B] length ab2_kv_save_row recorded, -1 none
-    size_t part_acc_bytes, part_ml_bytes;
+    size_t part_acc_bytes, part_ml_bytes, counter_bytes;
 };
 
 namespace ab2 {

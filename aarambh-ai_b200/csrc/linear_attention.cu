@@ -9,6 +9,11 @@
 //                                 o_i   = d^(i+1) S^T q_i + sum_{j <= i} d^(i-j) (q_i . k_j) v_j
 //                                 S_new = d^n S + sum_j d^(n-1-j) k_j v_j^T
 //
+// Where the heads of a prompt leave SMs idle it is cut into segments of whole chunks that run side by
+// side: a first launch (SUMS) forms every segment's own sum  sum_j d^(L-1-j) k_j v_j^T  and copies the
+// state before the prompt, the second starts each segment from those: with L the segment length,
+//     S_start(s) = d^(sL) S + sum_{r < s} d^((s-1-r)L) sum_r.
+//
 // q, k and v are bf16 as the projections leave them; everything else of the recurrence is f32.
 // Where an f32 quantity is an operand of a tensor-core product (the state, the decayed scores, the
 // decayed keys) it goes in as two bf16 terms, the rounded value and what rounding left, so the
@@ -117,7 +122,7 @@ __device__ __forceinline__ uint32_t tile_off(int r, int ch) {
 // grid (ceil(vdim / VS), H, rows), 4 warps.  A warp owns 16 tokens of the chunk's outputs and DP / 4 key
 // rows of the state's slice of VS value columns (accumulators in registers for the whole prompt; a
 // two-term copy in shared memory feeds the next chunk's product with the queries).
-template <int DP, int VS>
+template <int DP, int VS, bool SUMS>
 __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
     constexpr int C = LIGHTNING_CHUNK, MT = DP / 64, NV = VS / 8;
     constexpr int QB = C * DP * 2, VB = C * VS * 2, SB = DP * VS * 2, STAGE = 2 * QB + VB;
@@ -127,12 +132,17 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
     const int head = blockIdx.y, v0 = blockIdx.x * VS;
     const uint32_t sm = (uint32_t)__cvta_generic_to_shared(smem), s_hi = sm + 2 * STAGE, s_lo = s_hi + SB;
     for (int i = threadIdx.x; i <= C; i += 128) pw[i] = a.decay_pow[(size_t)head * (C + 1) + i];
+    const float pw_seg = a.decay_pow[(size_t)head * (C + 1) + C];
     pdl_wait();
     pdl_launch_dependents();
-    const int rrow = blockIdx.z, row = kv_row(a.kv, a.row0, rrow);
+    const int rrow = blockIdx.z / a.segs, seg = blockIdx.z % a.segs, row = kv_row(a.kv, a.row0, rrow);
+    const int seg0 = seg * a.seg_len, S_len = min(a.seg_len, a.S - seg0);  // tokens of this CTA
     float *state = a.kv.l.state + ((size_t)row * a.H + head) * a.dim * a.vdim;
+    // scratch slot r < segs - 1: segment r's own sum; slot segs - 1: the state before the prompt
+    const size_t slot_elems = (size_t)a.H * a.dim * a.vdim;
+    float *slots = a.scratch + (size_t)rrow * a.segs * slot_elems + (size_t)head * a.dim * a.vdim;
     const bool fresh = a.kv.lens[row] == 0;
-    const __nv_bfloat16 *base = (const __nv_bfloat16 *)a.qkv + (size_t)rrow * a.S * a.stride;
+    const __nv_bfloat16 *base = (const __nv_bfloat16 *)a.qkv + ((size_t)rrow * a.S + seg0) * a.stride;
     const __nv_bfloat16 *qb = base + (size_t)head * a.dim, *kb = qb + (size_t)a.H * a.dim;
     const __nv_bfloat16 *vb = base + 2 * (size_t)a.H * a.dim + (size_t)head * a.vdim + v0;
 
@@ -140,21 +150,22 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
         const uint32_t q = sm + buf * STAGE, k = q + QB, v = k + QB;
         for (int i = threadIdx.x; i < C * (DP / 8); i += 128) {
             const int r = i / (DP / 8), ch = i % (DP / 8);
-            const bool in = t0 + r < a.S && ch * 8 < a.dim;  // what is not there is zero
+            const bool in = t0 + r < S_len && ch * 8 < a.dim;  // what is not there is zero
             const size_t off = in ? (size_t)(t0 + r) * a.stride + ch * 8 : 0;
             const uint32_t d = tile_off<DP>(r, ch);
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(q + d), "l"(qb + off), "r"(in ? 16 : 0));
+            if (!SUMS) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(q + d), "l"(qb + off), "r"(in ? 16 : 0));
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(k + d), "l"(kb + off), "r"(in ? 16 : 0));
         }
         for (int i = threadIdx.x; i < C * (VS / 8); i += 128) {
             const int r = i / (VS / 8), ch = i % (VS / 8);
-            const bool in = t0 + r < a.S && v0 + ch * 8 < a.vdim;
+            const bool in = t0 + r < S_len && v0 + ch * 8 < a.vdim;
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(v + tile_off<VS>(r, ch)),
                          "l"(vb + (in ? (size_t)(t0 + r) * a.stride + ch * 8 : 0)), "r"(in ? 16 : 0));
         }
         asm volatile("cp.async.commit_group;\n" ::);
     };
-    load(0, 0);
+    const bool copies = SUMS && seg == a.segs - 1;  // this CTA hands on the state before the prompt
+    if (!copies) load(0, 0);
 
     float S[MT][NV][4];  // key rows (warp * MT + mt) * 16 + g, + 8; value columns n * 8 + 2c, + 1
 #pragma unroll
@@ -164,8 +175,25 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int d = (warp * MT + mt) * 16 + g + (j >> 1) * 8, v = v0 + n * 8 + 2 * c + (j & 1);
-                S[mt][n][j] = !fresh && d < a.dim && v < a.vdim ? state[(size_t)d * a.vdim + v] : 0.f;
+                const bool in = d < a.dim && v < a.vdim;
+                const size_t at = (size_t)d * a.vdim + v;
+                if (SUMS) S[mt][n][j] = copies && !fresh && in ? state[at] : 0.f;
+                else if (a.segs == 1) S[mt][n][j] = !fresh && in ? state[at] : 0.f;
+                else S[mt][n][j] = in ? slots[(size_t)(a.segs - 1) * slot_elems + at] : 0.f;
             }
+    if (!SUMS && seg > 0) {
+        const float dl = powf(pw_seg, (float)(a.seg_len / C));  // decay over a segment
+        for (int r = 0; r < seg; ++r)
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+                for (int n = 0; n < NV; ++n)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const int d = (warp * MT + mt) * 16 + g + (j >> 1) * 8, v = v0 + n * 8 + 2 * c + (j & 1);
+                        if (d < a.dim && v < a.vdim) S[mt][n][j] = fmaf(dl, S[mt][n][j], slots[(size_t)r * slot_elems + (size_t)d * a.vdim + v]);
+                    }
+    }
     auto publish = [&]() {
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
@@ -180,16 +208,17 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
                     asm volatile("st.shared.u32 [%0], %1;\n" ::"r"(s_lo + off), "r"(lo) : "memory");
                 }
     };
-    publish();
+    if (!SUMS) publish();
 
     int buf = 0;
-    for (int t0 = 0; t0 < a.S; t0 += C, buf ^= 1) {
-        const int n_tok = min(C, a.S - t0);
+    for (int t0 = 0; t0 < (copies ? 0 : S_len); t0 += C, buf ^= 1) {
+        const int n_tok = min(C, S_len - t0);
         asm volatile("cp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();  // this chunk's tiles and the state's copy are visible; the other buffers are free
-        if (t0 + C < a.S) load(t0 + C, buf ^ 1);
+        if (t0 + C < S_len) load(t0 + C, buf ^ 1);
         const uint32_t qs = sm + buf * STAGE, ks = qs + QB, vs = ks + QB;
 
+        if constexpr (!SUMS) {
         uint32_t qf[DP / 16][4];
 #pragma unroll
         for (int k = 0; k < DP / 16; ++k) ldsm4(qs + tile_off<DP>(warp * 16 + (lane & 15), k * 2 + (lane >> 4)), qf[k]);
@@ -257,10 +286,11 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
         for (int h = 0; h < 2; ++h) {
             const int i = h ? i1 : i0;
             if (i >= n_tok) continue;
-            float *dst = a.out + ((size_t)rrow * a.S + t0 + i) * a.H * a.vdim + (size_t)head * a.vdim + v0;
+            float *dst = a.out + ((size_t)rrow * a.S + seg0 + t0 + i) * a.H * a.vdim + (size_t)head * a.vdim + v0;
 #pragma unroll
             for (int n = 0; n < NV; ++n)
                 if (v0 + n * 8 + 2 * c < a.vdim) *reinterpret_cast<float2 *>(dst + n * 8 + 2 * c) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+        }
         }
         // the state after the chunk
         const float dn = pw[n_tok];
@@ -298,8 +328,10 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
             }
         }
         __syncthreads();  // every warp has read the state's copy
-        publish();
+        if (!SUMS) publish();
     }
+    if (!SUMS && seg != a.segs - 1) return;
+    float *end = SUMS ? slots + (size_t)seg * slot_elems : state;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -307,22 +339,45 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int d = (warp * MT + mt) * 16 + g + (j >> 1) * 8, v = v0 + n * 8 + 2 * c + (j & 1);
-                if (d < a.dim && v < a.vdim) state[(size_t)d * a.vdim + v] = S[mt][n][j];
+                if (d < a.dim && v < a.vdim) end[(size_t)d * a.vdim + v] = S[mt][n][j];
             }
 }
 
-template <int DP, int VS>
+template <int DP, int VS, bool SUMS>
 cudaError_t launch_chunk(const LightningArgs &a, int nrows, cudaStream_t s) {
     constexpr int smem = 2 * (2 * LIGHTNING_CHUNK * DP * 2 + LIGHTNING_CHUNK * VS * 2) + 2 * DP * VS * 2;
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev >= 0 && dev < 64 && !configured[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(lightning_chunk_kernel<DP, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(lightning_chunk_kernel<DP, VS, SUMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return e;
         configured[dev] = true;
     }
-    return launch_kernel(lightning_chunk_kernel<DP, VS>, dim3((a.vdim + VS - 1) / VS, a.H, nrows), dim3(128), (size_t)smem, s, a);
+    return launch_kernel(lightning_chunk_kernel<DP, VS, SUMS>, dim3((a.vdim + VS - 1) / VS, a.H, nrows * a.segs), dim3(128), (size_t)smem, s, a);
+}
+
+template <int DP, int VS>
+cudaError_t launch_prompt(const LightningArgs &a, int nrows, cudaStream_t s) {
+    if (a.segs > 1) {
+        cudaError_t e = launch_chunk<DP, VS, true>(a, nrows, s);
+        if (e != cudaSuccess) return e;
+    }
+    return launch_chunk<DP, VS, false>(a, nrows, s);
+}
+
+template <int DP>
+cudaError_t launch_prompt(LightningArgs a, int nrows, cudaStream_t s) {
+    // value slices of 64 columns, narrower ones while they leave SMs idle; then segments of at least four
+    // chunks, until there are two CTAs per SM
+    const int sms = device_sm_count();
+    auto ctas = [&](int vs) { return (a.vdim + vs - 1) / vs * a.H * nrows; };
+    const bool narrow = a.vdim <= 32 || (a.S < 8 * LIGHTNING_CHUNK && ctas(64) < sms);
+    int segs = std::min(LIGHTNING_MAX_SEGMENTS / std::max(1, nrows), std::min((2 * sms) / ctas(narrow ? 32 : 64), a.S / (4 * LIGHTNING_CHUNK)));
+    if (!a.scratch || segs < 2) segs = 1;
+    a.seg_len = ((a.S + segs - 1) / segs + LIGHTNING_CHUNK - 1) / LIGHTNING_CHUNK * LIGHTNING_CHUNK;
+    a.segs = (a.S + a.seg_len - 1) / a.seg_len;
+    return narrow ? launch_prompt<DP, 32>(a, nrows, s) : launch_prompt<DP, 64>(a, nrows, s);
 }
 
 // Prompts whose heads fit the chunk kernel; a handful of tokens is quicker one by one.
@@ -345,12 +400,7 @@ int lightning_attention(const LightningArgs &a, int nrows, ab2_dtype dtype, cuda
     cudaError_t e;
     if (dtype == AB2_F32) e = launch_serial<float>(a, nrows, s);
     else if (!chunk_eligible(a)) e = launch_serial<__nv_bfloat16>(a, nrows, s);
-    else {
-        // narrow value slices while the heads alone leave SMs idle
-        const bool narrow = a.vdim <= 32 || (long long)((a.vdim + 63) / 64) * a.H * nrows < device_sm_count();
-        if (a.dim <= 64) e = narrow ? launch_chunk<64, 32>(a, nrows, s) : launch_chunk<64, 64>(a, nrows, s);
-        else e = narrow ? launch_chunk<128, 32>(a, nrows, s) : launch_chunk<128, 64>(a, nrows, s);
-    }
+    else e = a.dim <= 64 ? launch_prompt<64>(a, nrows, s) : launch_prompt<128>(a, nrows, s);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "lightning attention launch failed: %s", cudaGetErrorString(e));
     return AB2_OK;
 }

@@ -360,9 +360,10 @@ __global__ void argmax_kernel(const T *__restrict__ logits, int vocab, uint32_t 
     __shared__ long long warp_best[32];
     const T *row = logits + (size_t)blockIdx.x * vocab;
     long long best = LLONG_MIN;
-    if (sizeof(T) == 2 && ((uintptr_t)row & 15) == 0) {
-        // 16-bit logits: eight per load, every load of a thread in flight at once
-        const int nvec = vocab >> 3;
+    if (((uintptr_t)row & 15) == 0) {
+        // 16 bytes of logits per load, every load of a thread in flight at once
+        constexpr int V = 16 / sizeof(T);
+        const int nvec = vocab / V;
         const uint4 *row4 = reinterpret_cast<const uint4 *>(row);
         for (int i0 = threadIdx.x; i0 < nvec; i0 += 4 * blockDim.x) {
             uint4 v[4];
@@ -377,10 +378,10 @@ __global__ void argmax_kernel(const T *__restrict__ logits, int vocab, uint32_t 
                 if (i >= nvec) continue;
                 const T *e = reinterpret_cast<const T *>(&v[u]);
 #pragma unroll
-                for (int j = 0; j < 8; ++j) best = max(best, argmax_key(to_f32(e[j]), i * 8 + j));
+                for (int j = 0; j < V; ++j) best = max(best, argmax_key(to_f32(e[j]), i * V + j));
             }
         }
-        for (int i = (nvec << 3) + threadIdx.x; i < vocab; i += blockDim.x) best = max(best, argmax_key(to_f32(row[i]), i));
+        for (int i = nvec * V + threadIdx.x; i < vocab; i += blockDim.x) best = max(best, argmax_key(to_f32(row[i]), i));
     } else {
         for (int i = threadIdx.x; i < vocab; i += blockDim.x) best = max(best, argmax_key(to_f32(row[i]), i));
     }

@@ -42,7 +42,7 @@ struct Stack {
     float *x, *mix32, *parts, *router_z;
     void *xb, *proj, *mixed, *act, *gathered, *v_first, *head_in;
     int *route_int;
-    float *route_score, *logits_scratch;
+    float *route_score, *logits_scratch, *seg_states;
     bool ready;
 };
 
@@ -100,7 +100,7 @@ int stack_create(Stack **out, const ab2_model_config &cfg, const ab2_layer_spec 
 static void free_workspace(Stack *st) {
     void **all[] = {(void **)&st->x, (void **)&st->mix32, (void **)&st->parts, (void **)&st->router_z, &st->xb, &st->proj, &st->mixed,
                     &st->act, &st->gathered, &st->v_first, &st->head_in, (void **)&st->route_int, (void **)&st->route_score,
-                    (void **)&st->logits_scratch};
+                    (void **)&st->logits_scratch, (void **)&st->seg_states};
     for (void **p : all) { cudaFree(*p); *p = nullptr; }
 }
 
@@ -189,7 +189,7 @@ int stack_finalize(Stack *st) {
         AB2_REQUIRE(st->cfg.tied, AB2_ERR_BAD_ARG, "lm_head not set and embeddings are not tied");
         st->lm_head = st->embedding;
     }
-    size_t proj = 0, mixed = 0, mix32 = 0, parts = 1, act = 0, gathered = 0, z = 0, vf = 0, pairs = 0, experts = 0;
+    size_t proj = 0, mixed = 0, mix32 = 0, parts = 1, act = 0, gathered = 0, z = 0, vf = 0, pairs = 0, experts = 0, state = 0;
     for (int i = 0; i < st->cfg.n_layers; ++i) {
         StackLayer &L = st->layers[i];
         const ab2_layer_spec &sp = L.spec;
@@ -200,6 +200,7 @@ int stack_finalize(Stack *st) {
         if (sp.mixer == AB2_MIX_LIGHTNING) {
             AB2_REQUIRE(L.mix_norm != nullptr, AB2_ERR_BAD_ARG, "layer %d: the mixer's norm is not set", i);
             mix32 = std::max(mix32, hv);
+            state = std::max(state, hv * sp.dim);
             std::vector<float> pw((size_t)sp.heads * (LIGHTNING_CHUNK + 1));
             for (int h = 0; h < sp.heads; ++h)
                 for (int n = 0; n <= LIGHTNING_CHUNK; ++n)
@@ -227,7 +228,8 @@ int stack_finalize(Stack *st) {
             {(void **)&st->mix32, T * mix32 * 4}, {(void **)&st->parts, T * parts * d * 4}, {&st->act, T * act * esz},
             {&st->gathered, b16 ? T * gathered * esz : 0}, {(void **)&st->router_z, T * z * 4}, {&st->v_first, T * vf * esz},
             {&st->head_in, T * d * esz}, {(void **)&st->route_int, (T * pairs * 2 + 2 * (experts + 1)) * 4},
-            {(void **)&st->route_score, T * pairs * 4}, {(void **)&st->logits_scratch, T * st->cfg.vocab * 4}};
+            {(void **)&st->route_score, T * pairs * 4}, {(void **)&st->logits_scratch, T * st->cfg.vocab * 4}, 
+            {(void **)&st->seg_states, b16 ? LIGHTNING_MAX_SEGMENTS * state * 4 : 0}};
         for (auto &a : all) {
             if (a.bytes == 0) continue;
             cudaError_t e = cudaMalloc(a.p, a.bytes);
@@ -266,9 +268,8 @@ static int attention_mixer(Stack *st, StackLayer &L, ab2_kv *kv, int layer, int 
     p.qkv = st->proj; p.stride = L.proj_width(); p.S = S; p.row0 = row0; p.H = sp.heads; p.G = sp.kv_heads; p.dim = sp.dim; p.vdim = sp.vdim;
     p.rot_dims = sp.rot_dims; p.qk_norm = sp.qk_norm; p.cos_t = L.cos_t; p.sin_t = L.sin_t; p.eps = st->cfg.rms_eps;
     p.v_first = st->v_first; p.v_mode = L.v_mode; p.lambda = sp.v_lambda;
-    STEP(window_prep(p, nrows, st->dtype, s));
     WindowAttnArgs a = {};
-    a.kv = p.kv; a.q = st->proj; a.q_stride = p.stride; a.out = st->mixed; a.S = S; a.row0 = row0; a.H = sp.heads;
+    a.prep = p; a.kv = p.kv; a.q = st->proj; a.q_stride = p.stride; a.out = st->mixed; a.S = S; a.row0 = row0; a.H = sp.heads;
     a.rep = sp.heads / sp.kv_heads; a.dim = sp.dim; a.vdim = sp.vdim; a.scale = sp.scale;
     return window_attention(kv, a, nrows, max_len, st->dtype, s);
 }
@@ -278,12 +279,12 @@ static int lightning_mixer(Stack *st, StackLayer &L, ab2_kv *kv, int layer, int 
     LightningArgs a = {};
     a.kv = kv_layer_view(kv, layer);
     a.qkv = st->proj; a.stride = L.proj_width(); a.out = st->mix32; a.S = S; a.row0 = row0; a.H = sp.heads; a.dim = sp.dim; a.vdim = sp.vdim;
-    a.decay_pow = L.decay_pow;
-    STEP(lightning_attention(a, nrows, st->dtype, s));
+    a.decay_pow = L.decay_pow; a.scratch = st->seg_states;
     ResidualNormArgs n = {};
     n.w = L.mix_norm; n.eps = st->cfg.rms_eps; n.d = sp.heads * sp.vdim; n.parts = st->mix32; n.out = st->mixed;
     n.gate = (const char *)st->proj + (size_t)sp.heads * (2 * sp.dim + sp.vdim) * dtype_size(st->dtype);
     n.gate_stride = a.stride;
+    STEP(lightning_attention(a, nrows, st->dtype, s));
     return launch_residual_norm(n, RN_GATED, nrows * S, st->dtype, s);
 }
 
@@ -391,9 +392,8 @@ AB2_API int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *sp
     p.S = S; p.row0 = row0; p.H = spec->heads; p.G = spec->kv_heads; p.dim = spec->dim; p.vdim = spec->vdim;
     p.rot_dims = spec->rot_dims; p.qk_norm = spec->qk_norm; p.cos_t = cos_dev; p.sin_t = sin_dev; p.eps = eps;
     p.v_first = v_first_dev; p.v_mode = v_mode; p.lambda = spec->v_lambda;
-    STEP(window_prep(p, nrows, dtype, (cudaStream_t)stream));
     WindowAttnArgs a = {};
-    a.kv = p.kv; a.q = qkv_dev; a.q_stride = p.stride; a.out = out_dev; a.S = S; a.row0 = row0; a.H = spec->heads;
+    a.prep = p; a.kv = p.kv; a.q = qkv_dev; a.q_stride = p.stride; a.out = out_dev; a.S = S; a.row0 = row0; a.H = spec->heads;
     a.rep = spec->heads / spec->kv_heads; a.dim = spec->dim; a.vdim = spec->vdim; a.scale = spec->scale;
     int max_len = 0;
     for (int i = 0; i < nrows; ++i) max_len = std::max(max_len, kv->lens_host[row0 + i] + S);
@@ -401,14 +401,14 @@ AB2_API int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *sp
 }
 
 AB2_API int ab2_lightning_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, const float *decay_pow_dev, const void *qkv_dev,
-                                    long long stride, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream) {
+                                    long long stride, float *scratch_dev, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream) {
     STEP(check_mixer_call(kv, layer, spec, AB2_MIX_LIGHTNING, qkv_dev, out_dev, S, row0, nrows, dtype));
     AB2_REQUIRE(decay_pow_dev != nullptr, AB2_ERR_BAD_ARG, "null decay table");
     AB2_REQUIRE(stride >= (long long)spec->heads * (2 * spec->dim + spec->vdim), AB2_ERR_BAD_SHAPE, "row stride %lld is too short", stride);
     LightningArgs a = {};
     a.kv = kv_layer_view(kv, layer);
     a.qkv = qkv_dev; a.stride = stride; a.out = out_dev; a.S = S; a.row0 = row0; a.H = spec->heads; a.dim = spec->dim; a.vdim = spec->vdim;
-    a.decay_pow = decay_pow_dev;
+    a.decay_pow = decay_pow_dev; a.scratch = scratch_dev;
     return lightning_attention(a, nrows, dtype, (cudaStream_t)stream);
 }
 

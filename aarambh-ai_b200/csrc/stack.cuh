@@ -22,6 +22,7 @@ struct WindowPrepArgs {
     float lambda;
 };
 struct WindowAttnArgs {
+    WindowPrepArgs prep;   // one token per row in bf16: done inside the attention kernel
     KvLayerView kv;
     const void *q;         // head h of token t at t * q_stride + h * dim
     long long q_stride;
@@ -29,10 +30,10 @@ struct WindowAttnArgs {
     int S, row0, H, rep, dim, vdim, nsplit;
     float scale;
     float *part_acc, *part_ml;
+    int *counters;         // [rows][G * head groups] split-arrival counters, 0 at rest
 };
-// Rotation, normalisation and value mixing of S new tokens per row, which are then stored in the cache.
-int window_prep(const WindowPrepArgs &a, int nrows, ab2_dtype dtype, cudaStream_t s);
-// Attention of the S tokens just stored; max_len bounds the rows' lengths with them.
+// Rotation, normalisation and value mixing of S new tokens per row, which are stored in the cache, and
+// their attention; max_len bounds the rows' lengths with them.  `a.prep` and `a` name the same tokens.
 int window_attention(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, ab2_dtype dtype, cudaStream_t s);
 
 // ---- lightning attention (linear_attention.cu) ------------------------------------
@@ -43,8 +44,11 @@ struct LightningArgs {
     float *out;            // [nrows * S][heads * vdim]
     int S, row0, H, dim, vdim;
     const float *decay_pow;  // [heads][LIGHTNING_CHUNK + 1]: powers 0, 1, ... of the head's decay
+    float *scratch;          // states of a prompt's segments: LIGHTNING_MAX_SEGMENTS x heads x dim x vdim, or null
+    int seg_len, segs;       // filled in by lightning_attention
 };
 constexpr int LIGHTNING_CHUNK = 64;
+constexpr int LIGHTNING_MAX_SEGMENTS = 16;  // over all rows of a call
 int lightning_attention(const LightningArgs &a, int nrows, ab2_dtype dtype, cudaStream_t s);
 
 // ---- normalisation around the f32 residual stream (ops.cu) -------------------------

@@ -156,14 +156,22 @@ def window_attention(cache, cfg, layer: int, qkv: torch.Tensor, tables, eps: flo
     return out
 
 
-def lightning_attention(cache, cfg, layer: int, qkv: torch.Tensor, powers: torch.Tensor, row0: int = 0) -> torch.Tensor:
+def lightning_scratch(cfg, layer: int) -> torch.Tensor:
+    """Scratch with which a long prompt of a lightning layer runs in segments side by side."""
+    m = cfg.layers[layer][0]
+    return torch.empty(16 * m.heads * m.dim * m.vdim, dtype=torch.float32, device="cuda")
+
+
+def lightning_attention(cache, cfg, layer: int, qkv: torch.Tensor, powers: torch.Tensor, row0: int = 0,
+                        scratch: torch.Tensor | None = None) -> torch.Tensor:
     """qkv [rows, S, stride] starting with heads dim | heads dim | heads vdim -> f32 [rows, S, heads vdim]."""
     qkv = _cuda(qkv, "qkv")
     specs, _keep = cfg.c_specs()
     sp = specs[layer]
     rows, S, stride = qkv.shape
     out = torch.empty((rows, S, sp.heads * sp.vdim), dtype=torch.float32, device=qkv.device)
-    check(lib.ab2_lightning_attention(cache._h, layer, C.byref(sp), powers.data_ptr(), qkv.data_ptr(), stride, out.data_ptr(), S, row0,
+    check(lib.ab2_lightning_attention(cache._h, layer, C.byref(sp), powers.data_ptr(), qkv.data_ptr(), stride,
+                                      scratch.data_ptr() if scratch is not None else None, out.data_ptr(), S, row0,
                                       rows, dtype_code(qkv.dtype), stream_ptr()))
     return out
 

@@ -275,9 +275,10 @@ int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void
                          const float *cos_dev, const float *sin_dev, float eps, void *out_dev, int S, int row0, int nrows,
                          ab2_dtype dtype, ab2_stream stream);
 /* Lightning attention: rows of qkv_dev hold q, k (heads dim each) and v (heads vdim), `stride` elements
- * apart; decay_pow_dev [heads][65] holds the powers 0..64 of each head's decay; out_dev [nrows * S][heads vdim] f32. */
+ * apart; decay_pow_dev [heads][65] holds the powers 0..64 of each head's decay; out_dev [nrows * S][heads vdim] f32.
+ * scratch_dev (16 * heads * dim * vdim floats, or NULL) lets a long prompt run in segments side by side. */
 int ab2_lightning_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, const float *decay_pow_dev, const void *qkv_dev,
-                            long long stride, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
+                            long long stride, float *scratch_dev, float *out_dev, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
 /* Mixture of experts: parts_dev [tokens][top][width] f32, the chosen experts' outputs (their sum is the
  * layer's).  Weights as in ab2_model_create_stack; workspace_dev holds ab2_moe_workspace bytes. */
 int ab2_moe_workspace(const ab2_layer_spec *spec, int width, int tokens, ab2_dtype dtype, size_t *bytes);

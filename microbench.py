@@ -373,8 +373,8 @@ def bench_stack(pkg, args):
             del caches
         for B, S in ((1, 512), (1, 2048), (1, 8192), (4, 2048)):
             cache = pkg.KVCache.for_stack(cfg, 1 << 20, B, 8192, "bf16")
-            qkv = x_of(B, S, 4 * H * 128)
-            t = time_graph(lambda: pkg.dispatch.lightning_attention(cache, cfg, 0, qkv, powers), 5, stream)
+            qkv, scratch = x_of(B, S, 4 * H * 128), pkg.dispatch.lightning_scratch(cfg, 0)
+            t = time_graph(lambda: pkg.dispatch.lightning_attention(cache, cfg, 0, qkv, powers, scratch=scratch), 5, stream)
             report("lightning_chunk_kernel", t, byt=B * S * H * 128 * (3 * 2 + 4), flops=B * S * H * 4.0 * 128 * 128, B=B, S=S)
             del cache
 

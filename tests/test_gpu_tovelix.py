@@ -184,6 +184,30 @@ def test_lightning_attention(dtype, H, dim, vdim, decay):
                 assert rel_err(got[:, h], want[:, h]) < tol(dtype, 2e-5, 1e-4), (sizes, h)
 
 
+@pytest.mark.parametrize("H,dim,vdim,T,rows", [(2, 64, 64, 1500, 1), (3, 128, 72, 700, 2), (1, 40, 24, 4100, 1)])
+def test_lightning_segments(H, dim, vdim, T, rows):
+    """Long prompts cut into segments that run side by side, on a row that already holds a state."""
+    p = pkg()
+    rng = np.random.default_rng(T)
+    decay = np.float32([0.9985, 0.6, 1.0][:H])
+    q, k, v = (fx.bf16_round(rng.standard_normal((rows, T, H, n)) * 0.3 + 0.1) for n in (dim, dim, vdim))
+    want = np.stack([ref.lightning_attention(q[r].astype(np.float64), k[r].astype(np.float64), v[r].astype(np.float64), decay.astype(np.float64))[0]
+                     for r in range(rows)])
+    qkv = to_gpu(np.concatenate([x.reshape(rows, T, -1) for x in (q, k, v)], 2), torch.bfloat16)
+    cfg = p.StackConfig(64, 64, [(p.LightningMixer(H, dim, vdim, decay.tolist()), None)], 2 * T)
+    powers, scratch = p.dispatch.decay_powers(decay.tolist()), p.dispatch.lightning_scratch(cfg, 0)
+    for cuts in ([0, T], [0, 19, T - 33, T], [0, 600, T]):
+        cache = p.KVCache.for_stack(cfg, 2 * T, rows, T, "bf16")
+        got = []
+        for a, b in zip(cuts, cuts[1:]):
+            got.append(p.dispatch.lightning_attention(cache, cfg, 0, qkv[:, a:b].contiguous(), powers, scratch=scratch))
+            cache.commit(b - a)
+        got = torch.cat(got, 1).cpu().numpy().reshape(want.shape)
+        for r in range(rows):
+            for h in range(H):
+                assert rel_err(got[r, :, h], want[r, :, h]) < 1e-4, (cuts, r, h)
+
+
 # ---------------------------------------------------------------- the model
 
 def tokens_of(n, vocab, seed):
