@@ -1,11 +1,15 @@
 """Tovelix on the GPU against the plain numpy restatement: every mechanism alone, then the model
 through its own cache, portions, batches, sessions and generation."""
+import json
+import os
+import subprocess
+
 import numpy as np
 import pytest
 import torch
 
 import tovelix_fixtures as fx
-from helpers import pkg, rel_err
+from helpers import ROOT, pkg, rel_err
 from oracle import tovelix_ref as ref
 from test_tovelix_host import spiked_attention
 
@@ -328,6 +332,41 @@ def test_greedy_generation(tmp_path):
             se.advance(s)
         se.decode_sessions([s for s in live if not s.finished])
     assert [s.generated_ids for s in live] == want
+
+
+def run_program(name, args, text=""):
+    exe = os.path.join(ROOT, "bin", name)
+    res = subprocess.run([exe, *args], input=text, capture_output=True, text=True, timeout=240)
+    assert res.returncode == 0, res.stderr[-2000:]
+    return res.stdout
+
+
+def test_command_line_programs(tmp_path):
+    """bin/generate and bin/trace_run on a checkpoint folder."""
+    cfg = fx.VARIED
+    w = fx.weights(cfg, 17)
+    folder = fx.write_checkpoint(str(tmp_path / "m"), cfg, w)
+    prompts = [tokens_of(n, cfg["vocab"], 50 + n) for n in (21, 3)]
+    want = [greedy(cfg, w, q, 5) for q in prompts]
+    base = ["--model", folder, "--dtype", "float32", "--max-new-tokens", "5"]
+    args = [["--tokens", ",".join(map(str, q))] for q in prompts]
+    one = run_program("generate", base + args[0])
+    two = run_program("generate", base + args[0] + args[1])
+    assert [json.loads(x)["tokens"] for x in one.splitlines()] == want[:1]
+    assert [json.loads(x)["tokens"] for x in two.splitlines()] == want
+    q = prompts[0]
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": q[:9], "want": [0, 8]}, {"id": "b", "tokens": q[:4], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": q[4:5], "want": [0]}], "end": ["b"]},
+             {"step": 2, "entries": [{"id": "a", "tokens": q[9:20], "want": []}], "end": []},
+             {"step": 3, "entries": [{"id": "a", "tokens": q[20:], "want": [0]}, {"id": "c", "tokens": q[:2], "want": [1]}], "end": ["a", "c"]}]
+    out = run_program("trace_run", ["--model", folder, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "40"],
+                      "\n".join(map(json.dumps, steps)) + "\n")
+    assert [x for x in out.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2", "done 3"]
+    full = fx.expected(cfg, w, q)
+    for step, at in ((0, [0, 8]), (1, [4]), (3, [20, 1])):
+        got = np.fromfile(tmp_path / f"{step}.f32", "<f4").reshape(len(at), cfg["vocab"])
+        check_logits(got.astype(np.float64), full[at], torch.float32)
+    assert not (tmp_path / "2.f32").exists()
 
 
 def test_draft_verification_restores_the_state(tmp_path):
