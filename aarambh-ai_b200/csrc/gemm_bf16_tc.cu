@@ -12,7 +12,7 @@
 //   warp 1     MMA issue (one elected thread); accumulators in tensor memory, two sets, so that the
 //              epilogue of a tile overlaps the MMAs of the next.  MOE_GLU keeps a gate and an up
 //              accumulator per set, lane for lane, so the gated unit needs no exchange.
-//   warps 2-5  epilogue: tcgen05.ld, epilogue arithmetic in f32, stores.
+//   warps 2-9  epilogue: tcgen05.ld, epilogue arithmetic in f32, stores.
 // The tiles of the grouped modes follow from the device-side expert offsets: every CTA lays the
 // same tile list out from them (prefix sums in shared memory).  Rows of a tile past its expert's
 // last pair belong to the next expert; they are multiplied and not stored.  The pair's weight
@@ -35,7 +35,8 @@ int device_status_word(int **out);
 int device_sm_count();
 namespace {
 
-constexpr int GB_THREADS = 192;
+constexpr int GB_EPI_WARPS = 8;  // two per tensor-memory quadrant: they take alternate token blocks
+constexpr int GB_THREADS = 64 + GB_EPI_WARPS * 32;
 constexpr int GB_A_BYTES = 128 * 128;  // 128 channels x 64 bf16
 constexpr int GB_MAX_STAGES = 8;
 constexpr int GB_MAX_EXPERTS = 1024;
@@ -89,7 +90,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
 
     if (threadIdx.x == 0) {
         for (int i = 0; i < STAGES; ++i) { bar_init(&sh->full[i], 1); bar_init(&sh->empty[i], 1); }
-        for (int i = 0; i < 2; ++i) { bar_init(&sh->accfull[i], 1); bar_init(&sh->accempty[i], 4); }
+        for (int i = 0; i < 2; ++i) { bar_init(&sh->accfull[i], 1); bar_init(&sh->accempty[i], GB_EPI_WARPS); }
         sh->failed = 0;
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
@@ -177,7 +178,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
         }
     } else {
         // ---------------------------------------------------------- epilogue
-        const int quad = warp & 3;
+        const int quad = warp & 3, first_block = (warp - 2) >> 2;
         uint32_t tuse = 0;
         for (int it = blockIdx.x; it < items && !*failed; it += gridDim.x, ++tuse) {
             int nt, mt;
@@ -191,7 +192,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
             const int n = nt * 128 + quad * 32 + lane;
             constexpr int CW = DUAL ? 16 : 32;  // tokens per register block
 #pragma unroll 1
-            for (int c = 0; c < NTOK / CW; ++c) {
+            for (int c = first_block; c < NTOK / CW; c += GB_EPI_WARPS / 4) {
                 __syncwarp();  // the tensor-memory load is a whole-warp operation
                 if (c * CW >= cnt) break;
                 const uint32_t taddr = tmem + ((uint32_t)(quad * 32) << 16) + (uint32_t)(ab * ACC_COLS + c * CW);
@@ -231,7 +232,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                         for (int j = 0; j < CW; ++j) {
                             float f = __uint_as_float(v[j]);
                             if (act) {
-                                const float sg = 1.f / (1.f + __expf(-f));
+                                const float sg = __fdividef(1.f, 1.f + __expf(-f));
                                 f = silu ? f * sg : sg;
                             }
                             if (c * CW + j < cnt) y[(size_t)j * a.N] = __float2bfloat16_rn(f);

@@ -10,9 +10,9 @@
 //                                 S_new = d^n S + sum_j d^(n-1-j) k_j v_j^T
 //
 // Where the heads of a prompt leave SMs idle it is cut into segments of whole chunks that run side by
-// side: a first launch (SUMS) forms every segment's own sum  sum_j d^(L-1-j) k_j v_j^T  and copies the
-// state before the prompt, the second starts each segment from those: with L the segment length,
-//     S_start(s) = d^(sL) S + sum_{r < s} d^((s-1-r)L) sum_r.
+// side: a first launch (SUMS) forms every segment's own sum  sum_j d^(L-1-j) k_j v_j^T  (L the segment
+// length) and copies the state before the prompt, a second (lightning_scan_kernel) makes the state before
+// each segment of them,  S_(r+1) = d^L S_r + sum_r,  and the third computes the outputs.
 //
 // q, k and v are bf16 as the projections leave them; everything else of the recurrence is f32.
 // Where an f32 quantity is an operand of a tensor-core product (the state, the decayed scores, the
@@ -132,13 +132,13 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
     const int head = blockIdx.y, v0 = blockIdx.x * VS;
     const uint32_t sm = (uint32_t)__cvta_generic_to_shared(smem), s_hi = sm + 2 * STAGE, s_lo = s_hi + SB;
     for (int i = threadIdx.x; i <= C; i += 128) pw[i] = a.decay_pow[(size_t)head * (C + 1) + i];
-    const float pw_seg = a.decay_pow[(size_t)head * (C + 1) + C];
     pdl_wait();
     pdl_launch_dependents();
     const int rrow = blockIdx.z / a.segs, seg = blockIdx.z % a.segs, row = kv_row(a.kv, a.row0, rrow);
     const int seg0 = seg * a.seg_len, S_len = min(a.seg_len, a.S - seg0);  // tokens of this CTA
     float *state = a.kv.l.state + ((size_t)row * a.H + head) * a.dim * a.vdim;
-    // scratch slot r < segs - 1: segment r's own sum; slot segs - 1: the state before the prompt
+    // scratch slots: from SUMS segment r's own sum (r < segs - 1) and the state before the prompt (the last),
+    // after lightning_scan_kernel the state before segment r
     const size_t slot_elems = (size_t)a.H * a.dim * a.vdim;
     float *slots = a.scratch + (size_t)rrow * a.segs * slot_elems + (size_t)head * a.dim * a.vdim;
     const bool fresh = a.kv.lens[row] == 0;
@@ -179,21 +179,8 @@ __global__ void __launch_bounds__(128) lightning_chunk_kernel(LightningArgs a) {
                 const size_t at = (size_t)d * a.vdim + v;
                 if (SUMS) S[mt][n][j] = copies && !fresh && in ? state[at] : 0.f;
                 else if (a.segs == 1) S[mt][n][j] = !fresh && in ? state[at] : 0.f;
-                else S[mt][n][j] = in ? slots[(size_t)(a.segs - 1) * slot_elems + at] : 0.f;
+                else S[mt][n][j] = in ? slots[(size_t)seg * slot_elems + at] : 0.f;
             }
-    if (!SUMS && seg > 0) {
-        const float dl = powf(pw_seg, (float)(a.seg_len / C));  // decay over a segment
-        for (int r = 0; r < seg; ++r)
-#pragma unroll
-            for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-                for (int n = 0; n < NV; ++n)
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        const int d = (warp * MT + mt) * 16 + g + (j >> 1) * 8, v = v0 + n * 8 + 2 * c + (j & 1);
-                        if (d < a.dim && v < a.vdim) S[mt][n][j] = fmaf(dl, S[mt][n][j], slots[(size_t)r * slot_elems + (size_t)d * a.vdim + v]);
-                    }
-    }
     auto publish = [&]() {
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
@@ -357,10 +344,35 @@ cudaError_t launch_chunk(const LightningArgs &a, int nrows, cudaStream_t s) {
     return launch_kernel(lightning_chunk_kernel<DP, VS, SUMS>, dim3((a.vdim + VS - 1) / VS, a.H, nrows * a.segs), dim3(128), (size_t)smem, s, a);
 }
 
+// grid (blocks over a head's state, H, rows): the slots of one state element, in order.
+__global__ void __launch_bounds__(256) lightning_scan_kernel(LightningArgs a) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int n = a.dim * a.vdim, i = blockIdx.x * 256 + threadIdx.x;
+    if (i >= n) return;
+    float *slot = a.scratch + (size_t)blockIdx.z * a.segs * a.H * n + (size_t)blockIdx.y * n + i;
+    const size_t step = (size_t)a.H * n;
+    const float dl = powf(a.decay_pow[(size_t)blockIdx.y * (LIGHTNING_CHUNK + 1) + LIGHTNING_CHUNK], (float)(a.seg_len / LIGHTNING_CHUNK));
+    float v[LIGHTNING_MAX_SEGMENTS];
+#pragma unroll
+    for (int r = 0; r < LIGHTNING_MAX_SEGMENTS; ++r) v[r] = r < a.segs ? slot[r * step] : 0.f;
+    float S = 0.f;
+#pragma unroll
+    for (int r = 0; r < LIGHTNING_MAX_SEGMENTS; ++r)
+        if (r == a.segs - 1) S = v[r];
+#pragma unroll
+    for (int r = 0; r < LIGHTNING_MAX_SEGMENTS; ++r) {
+        if (r < a.segs) slot[r * step] = S;
+        S = fmaf(dl, S, v[r]);
+    }
+}
+
 template <int DP, int VS>
 cudaError_t launch_prompt(const LightningArgs &a, int nrows, cudaStream_t s) {
     if (a.segs > 1) {
         cudaError_t e = launch_chunk<DP, VS, true>(a, nrows, s);
+        if (e == cudaSuccess)
+            e = launch_kernel(lightning_scan_kernel, dim3((a.dim * a.vdim + 255) / 256, a.H, nrows), dim3(256), 0, s, a);
         if (e != cudaSuccess) return e;
     }
     return launch_chunk<DP, VS, false>(a, nrows, s);

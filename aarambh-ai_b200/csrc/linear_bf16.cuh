@@ -47,7 +47,7 @@ struct LinArgs {
 // g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)
 __device__ __forceinline__ float clamped_glu_value(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+    return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
 }
 __device__ __forceinline__ float clamped_glu_value_exact(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
