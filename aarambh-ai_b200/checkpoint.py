@@ -1,5 +1,5 @@
-"""Reader of safetensors files: an 8-byte little-endian length, that many bytes of JSON
-(name -> dtype, shape, data_offsets), then the data."""
+"""Reader of safetensors files.  Their header is a u64 size and a JSON table that gives every
+tensor's element type, shape and byte range in the payload behind it."""
 from __future__ import annotations
 
 import json

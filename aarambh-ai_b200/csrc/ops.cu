@@ -215,6 +215,30 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
     const T *gate = (const T *)a.gate + t * (size_t)a.gate_stride;
     float *x = a.x + t * (size_t)a.d;
     // a thread reads back the elements it wrote, so the row needs no second barrier
+    if (vec && (MODE != RN_GATED || ((uintptr_t)gate & (4 * sizeof(T) - 1)) == 0)) {
+        for (int i = threadIdx.x; i < a.d / 4; i += blockDim.x) {
+            const float4 r = reinterpret_cast<const float4 *>(vrow)[i], w = reinterpret_cast<const float4 *>(a.w)[i];
+            float v[4] = {r.x * inv * w.x, r.y * inv * w.y, r.z * inv * w.z, r.w * inv * w.w};
+            struct alignas(4 * sizeof(T)) Quad { T e[4]; };
+            if (MODE == RN_ADD) {
+                const float4 q = reinterpret_cast<const float4 *>(x)[i];
+                v[0] += q.x; v[1] += q.y; v[2] += q.z; v[3] += q.w;
+            }
+            if (MODE == RN_GATED) {
+                const Quad q = reinterpret_cast<const Quad *>(gate)[i];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) v[j] *= to_f32(q.e[j]);
+            }
+            if (MODE == RN_EMBED || MODE == RN_ADD) reinterpret_cast<float4 *>(x)[i] = make_float4(v[0], v[1], v[2], v[3]);
+            if (a.out != nullptr) {
+                Quad q;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) q.e[j] = from_f32<T>(v[j]);
+                reinterpret_cast<Quad *>(out)[i] = q;
+            }
+        }
+        return;
+    }
     const int step = vec ? 4 : 1;
     for (int i0 = threadIdx.x * step; i0 < a.d; i0 += blockDim.x * step) {
         for (int j = 0; j < step; ++j) {

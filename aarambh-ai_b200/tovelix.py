@@ -1,7 +1,8 @@
-"""Tovelix: a decoder of sliding-window attention layers (rotation, then q and k on unit root
-mean square; values mixed with those of the first such layer) and lightning-attention layers,
-each with a mixture of experts whose router scores multiply the experts' inputs; norms on the
-sublayers' outputs only; tied embeddings with a norm of their own.
+"""Tovelix: a decoder that mixes layers of sliding-window attention (q and k rotated, then scaled to
+unit RMS; values blended with those of the first layer that does so) and of lightning attention, with
+sparse experts whose router scores scale what an expert reads.  The residual stream enters every
+sublayer unnormalised and each sublayer's result is RMS-normed before it is added; the head is the
+embedding table.
 
 This module maps a checkpoint folder (config.json, model.safetensors) to a ``StackConfig`` and
 its weights; the layers themselves are those of ``StackModel``.

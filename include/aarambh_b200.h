@@ -267,8 +267,8 @@ int ab2_kv_read(const ab2_kv *kv, int layer, int row, float *k_out_dev, float *v
 /* ---- mechanisms of layer stacks as operators ---------------------------------------
  * Each works on one layer of a stack cache at the rows' current lengths, which it does not advance
  * (ab2_kv_commit does, once every layer has run).
- * Window attention: qkv_dev [nrows * S][heads dim | kv_heads dim | kv_heads vdim], the queries are
- * rewritten; rotation and normalisation as the spec says (tables [positions][rot_dims / 2]); v_mode 1
+ * Window attention: qkv_dev [nrows * S][heads dim | kv_heads dim | kv_heads vdim], the queries may be
+ * rewritten in place; rotation and normalisation as the spec says (tables [positions][rot_dims / 2]); v_mode 1
  * copies the values to v_first_dev [nrows * S][kv_heads vdim], 2 mixes them with it; out_dev
  * [nrows * S][heads vdim]. */
 int ab2_window_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *qkv_dev, void *v_first_dev, int v_mode,

@@ -379,9 +379,35 @@ def bench_stack(pkg, args):
             del cache
 
 
+def run_stack_step(pkg, args):
+    """Three graph-replayed decode steps (context 512, --batch sequences) or two prefills of --prompt tokens of
+    a Tovelix stack of bench.py's size --size with the layers --pattern: the workload of the stack's profiles."""
+    import bench
+    c = dict(bench.TOVELIX[args.size], layers=args.pattern)
+    B, S = (1, args.prompt) if args.prompt else (args.batch, 512)
+    model = bench.build_tovelix(pkg, torch, c, max(S, 32), S + 64)
+    cache = model.empty_kv_cache_with_capacity(S + 40, batch=B)
+    prompt = torch.randint(0, 32000, (B, S), generator=torch.Generator().manual_seed(1))
+    stream = torch.cuda.Stream()
+    with torch.cuda.stream(stream):
+        if args.prompt:
+            for _ in range(2):
+                cache.truncate(0, 0)
+                model.forward_with_cache(prompt, 0, cache, row=0, last_only=True)
+        else:
+            logits = torch.cat([model.forward_with_cache(prompt[b:b + 1], 0, cache, row=b, last_only=True).view(1, -1) for b in range(B)])
+            bufs = [pkg.dispatch.argmax(logits).clone(), torch.empty(B, dtype=torch.int32, device="cuda")]
+            for i in range(3):
+                model.decode_step(bufs[i % 2], cache, None, bufs[(i + 1) % 2])
+    stream.synchronize()
+
+
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("what", choices=["gemv", "gemm", "attention", "prefill_attention", "step", "stack"])
+    ap.add_argument("what", choices=["gemv", "gemm", "attention", "prefill_attention", "step", "stack", "stack_step"])
+    ap.add_argument("--size", default="w2048", help="stack_step: a size of bench.py's Tovelix table")
+    ap.add_argument("--pattern", default="LA", help="stack_step: layers, L lightning, A attention")
+    ap.add_argument("--prompt", type=int, default=0, help="stack_step: prefill this many tokens (0: decode steps)")
     ap.add_argument("--only", default=None, help="stack: linear, moe, window, lightning")
     ap.add_argument("--layers", type=int, default=2)
     ap.add_argument("--ctx", type=int, default=512)
@@ -405,6 +431,8 @@ def main():
         bench_gemm(pkg, args)
     elif args.what == "step":
         bench_step(pkg, args)
+    elif args.what == "stack_step":
+        run_stack_step(pkg, args)
     elif args.what == "stack":
         bench_stack(pkg, args)
     elif args.what == "prefill_attention":

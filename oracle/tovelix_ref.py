@@ -16,7 +16,7 @@ import numpy as np
 
 
 def rms(x, eps):
-    """x divided by its root mean square over the last axis, eps inside the root."""
+    """x / sqrt(mean(x^2) + eps) along the last axis."""
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + x.dtype.type(eps))
 
 
