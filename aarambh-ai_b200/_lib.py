@@ -89,12 +89,18 @@ SIGNATURES = {
     "ab2_lightning_attention": ([_p, _i, _p, _p, _p, C.c_longlong, _p, _p, _i, _i, _i, _i, _p], _i),
     "ab2_moe_workspace": ([_p, _i, _i, _i, C.POINTER(C.c_size_t)], _i),
     "ab2_moe_forward": ([_p, _p, _p, _p, _p, _p, _i, _i, _p, _p, _p], _i),
+    "ab2_latent_workspace": ([_p, _i, _i, _i, C.POINTER(C.c_size_t)], _i),
+    "ab2_latent_attention": ([_p, _i, _p, _p, C.c_longlong, _p, _p, _p, _p, _f, _p, _p, C.c_size_t, _i, _i, _i, _i, _p], _i),
+    "ab2_poly_norm": ([_p, _p, _i, _i, C.POINTER(_f), _f, _i, _p], _i),
     "ab2_attention_decode": ([_p, _i, _p, _p, _i, _i, _f, _i, _p], _i),
     "ab2_attention_decode_static": ([_p, _i, _p, _p, _i, _i, _f, _i, _p], _i),
     "ab2_attention_cached": ([_p, _i, _p, _p, _i, _i, _i, _f, _i, _p], _i),
     "ab2_attention_causal": ([_p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _p], _i),
     "ab2_model_create": ([_pp, _p, _i, _i], _i),
     "ab2_model_create_stack": ([_pp, _p, _p, _i, _i], _i),
+    "ab2_model_set_form": ([_p, _p], _i),
+    "ab2_model_set_loop_steps": ([_p, _p], _i),
+    "ab2_model_set_expert_table": ([_p, _i, _p], _i),
     "ab2_model_destroy": ([_p], _i),
     "ab2_model_set_linear": ([_p, _i, _i, _p], _i),
     "ab2_model_set_norm": ([_p, _i, _i, _p], _i),
@@ -129,8 +135,10 @@ class ModelConfig(C.Structure):
                 ("rms_eps", _f), ("rope_theta", C.c_double), ("tied", _i)]
 
 
-MIX_ATTENTION, MIX_LIGHTNING = 0, 1
-FFN_NONE, FFN_MOE = 0, 1
+MIX_ATTENTION, MIX_LIGHTNING, MIX_LATENT = 0, 1, 2
+FFN_NONE, FFN_MOE, FFN_POLY = 0, 1, 2
+GLU = {"clamped": 0, "silu": 1}
+ROUTING = {"sigmoid": 0, "table": 1}
 
 
 class LayerSpec(C.Structure):
@@ -138,7 +146,12 @@ class LayerSpec(C.Structure):
     _fields_ = [("mixer", _i), ("heads", _i), ("dim", _i), ("vdim", _i), ("kv_heads", _i), ("window", _i),
                 ("rot_dims", _i), ("rot_base", C.c_double), ("qk_norm", _i), ("scale", _f), ("v_mix", _i),
                 ("v_lambda", _f), ("decay", C.POINTER(_f)), ("ffn", _i), ("experts", _i), ("top", _i), ("ff", _i),
-                ("limit", _f)]
+                ("limit", _f), ("kv_rank", _i), ("head_gate", _i), ("glu", _i), ("routing", _i), ("shared_ff", _i), ("poly", _f * 4)]
+
+
+class StackForm(C.Structure):
+    """ab2_stack_form."""
+    _fields_ = [("embed_norm", _i), ("pre_norms", _i), ("loop_start", _i), ("loop_stop", _i), ("loop_times", _i), ("logit_softcap", _f)]
 
 
 def _declare():

@@ -6,7 +6,7 @@
 //                              root mean square, value mixing, store into the ring
 //   window_attn_kernel         f32 arithmetic on CUDA cores: decode (the window split over CTAs,
 //                              log-sum-exp merge), f32 models, unusual head sizes
-//   window_attn_mma_kernel     prompts in bf16 on the warp-level tensor cores
+//   window_attn_mma_kernel     prompts in bf16 on the warp-level tensor cores; also over explicit keys (prompt_attention)
 //   window_decode_mma_kernel   decode in bf16, preparation included, on the warp-level tensor cores
 //
 // Scores, softmax weights and sums are f32 throughout.  The tensor-core kernel multiplies the
@@ -14,6 +14,7 @@
 // product carries them to about 16 significant bits instead of 8.
 #include <algorithm>
 #include <cfloat>
+#include <type_traits>
 
 #include "stack.cuh"
 
@@ -267,37 +268,56 @@ __device__ __forceinline__ void split_pair(float x, float y, uint32_t &hi, uint3
     lo = (uint32_t)__bfloat16_as_ushort(xl) | ((uint32_t)__bfloat16_as_ushort(yl) << 16);
 }
 
-template <int DP, int VP>
-__global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) {
+// The keys come from a stack cache (WindowAttnArgs: grid z is the row) or lie position by position with
+// the last `tail_dims` dimensions in a matrix of their own (PromptAttnArgs).
+template <int DP, int VP, class Args>
+__global__ void __launch_bounds__(128) window_attn_mma_kernel(Args a) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int KT = 64, KB = KT * DP * 2, VB = KT * VP * 2;
+    constexpr bool EXPLICIT = std::is_same<Args, PromptAttnArgs>::value;
     pdl_wait();
     pdl_launch_dependents();
-    const KvLayer &l = a.kv.l;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
-    const int head = blockIdx.y, kvh = head / a.rep, rrow = blockIdx.z, row = kv_row(a.kv, a.row0, rrow);
+    const int head = blockIdx.y, rrow = blockIdx.z;
     const int q_lo = ((int)gridDim.x - 1 - (int)blockIdx.x) * 64;  // the longest key walks first
-    const int len = a.kv.lens[row];
-    const __nv_bfloat16 *kb = (const __nv_bfloat16 *)l.k + ((size_t)row * l.kvh + kvh) * l.cap * l.kds;
-    const __nv_bfloat16 *vb = (const __nv_bfloat16 *)l.v + ((size_t)row * l.kvh + kvh) * l.cap * l.vds;
-    const int key_lo = max(0, len + q_lo - l.window + 1), key_hi = len + min(a.S, q_lo + 64) - 1;
+    const __nv_bfloat16 *kb, *vb, *tail = nullptr, *q0;
+    size_t kst, vst, tst = 0, out_stride;
+    int len, window, cap, dim, kdims, vdims, kmain;  // key dimensions from kmain on are in `tail`
+    if constexpr (EXPLICIT) {
+        kb = a.k + (size_t)head * a.k_head; vb = a.v + (size_t)head * a.v_head; tail = a.tail;
+        kst = a.k_stride; vst = a.v_stride; tst = a.tail_stride;
+        len = a.first; window = 1 << 30; cap = 1 << 30;
+        dim = kdims = a.dim + a.tail_dims; kmain = a.dim; vdims = a.vdim;
+        q0 = a.q + (size_t)head * dim; out_stride = a.out_stride;
+    } else {
+        const KvLayer &l = a.kv.l;
+        const int kvh = head / a.rep, row = kv_row(a.kv, a.row0, rrow);
+        kb = (const __nv_bfloat16 *)l.k + ((size_t)row * l.kvh + kvh) * l.cap * l.kds;
+        vb = (const __nv_bfloat16 *)l.v + ((size_t)row * l.kvh + kvh) * l.cap * l.vds;
+        kst = l.kds; vst = l.vds;
+        len = a.kv.lens[row]; window = l.window; cap = l.cap;
+        dim = a.dim; kdims = kmain = l.kds; vdims = l.vds;
+        q0 = (const __nv_bfloat16 *)a.q + (size_t)rrow * a.S * a.q_stride + (size_t)head * dim; out_stride = (size_t)a.H * a.vdim;
+    }
+    const int key_lo = max(0, len + q_lo - window + 1), key_hi = len + min(a.S, q_lo + 64) - 1;
 
     auto load_tile = [&](int base, int buf) {
         const uint32_t ks = (uint32_t)__cvta_generic_to_shared(smem) + buf * (KB + VB), vs = ks + KB;
-        const int slot0 = base % l.cap;
+        const int slot0 = EXPLICIT ? base : base % cap;
         for (int i = threadIdx.x; i < KT * (DP / 8); i += 128) {
             const int r = i / (DP / 8), ch = i % (DP / 8);
             int slot = slot0 + min(r, key_hi - base);  // rows past the last key repeat it (masked below)
-            if (slot >= l.cap) slot -= l.cap;
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(ks + r * DP * 2 + ((ch ^ (r & 7)) << 4)),
-                         "l"(kb + (size_t)slot * l.kds + (ch * 8 < l.kds ? ch * 8 : 0)), "r"(ch * 8 < l.kds ? 16 : 0));
+            if (!EXPLICIT && slot >= cap) slot -= cap;
+            const __nv_bfloat16 *src = EXPLICIT && ch * 8 >= kmain && ch * 8 < kdims ? tail + slot * tst + (ch * 8 - kmain)
+                                                                                      : kb + slot * kst + (ch * 8 < kdims ? ch * 8 : 0);
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(ks + r * DP * 2 + ((ch ^ (r & 7)) << 4)), "l"(src), "r"(ch * 8 < kdims ? 16 : 0));
         }
         for (int i = threadIdx.x; i < KT * (VP / 8); i += 128) {
             const int r = i / (VP / 8), ch = i % (VP / 8);
             int slot = slot0 + min(r, key_hi - base);
-            if (slot >= l.cap) slot -= l.cap;
+            if (!EXPLICIT && slot >= cap) slot -= cap;
             asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(vs + r * VP * 2 + ((ch ^ (r & 7)) << 4)),
-                         "l"(vb + (size_t)slot * l.vds + (ch * 8 < l.vds ? ch * 8 : 0)), "r"(ch * 8 < l.vds ? 16 : 0));
+                         "l"(vb + slot * vst + (ch * 8 < vdims ? ch * 8 : 0)), "r"(ch * 8 < vdims ? 16 : 0));
         }
         asm volatile("cp.async.commit_group;\n" ::);
     };
@@ -307,14 +327,14 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
     const int pa = len + qa, pb = len + qb;  // positions of this thread's two rows
     uint32_t qf[DP / 16][4];
     {
-        const __nv_bfloat16 *ra = (const __nv_bfloat16 *)a.q + ((size_t)rrow * a.S + min(qa, a.S - 1)) * a.q_stride + (size_t)head * a.dim;
-        const __nv_bfloat16 *rb = (const __nv_bfloat16 *)a.q + ((size_t)rrow * a.S + min(qb, a.S - 1)) * a.q_stride + (size_t)head * a.dim;
+        const __nv_bfloat16 *ra = q0 + (size_t)min(qa, a.S - 1) * a.q_stride;
+        const __nv_bfloat16 *rb = q0 + (size_t)min(qb, a.S - 1) * a.q_stride;
 #pragma unroll
         for (int ks = 0; ks < DP / 16; ++ks)
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
                 const int d = ks * 16 + h * 8 + 2 * c;
-                const bool in = d < a.dim;
+                const bool in = d < dim;
                 qf[ks][2 * h] = in ? *reinterpret_cast<const uint32_t *>(ra + d) : 0u;
                 qf[ks][2 * h + 1] = in ? *reinterpret_cast<const uint32_t *>(rb + d) : 0u;
             }
@@ -335,7 +355,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
         else asm volatile("cp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();
         const uint32_t ks0 = (uint32_t)__cvta_generic_to_shared(smem) + buf * (KB + VB), vs0 = ks0 + KB;
-        if (base <= w_last && base + KT - 1 > w_first - l.window) {
+        if (base <= w_last && base + KT - 1 > w_first - window) {
             float s[8][4];
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {
@@ -352,7 +372,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
                     mma_bf16(s[nt], qf[2 * k2 + 1], b2, b3);
                 }
             }
-            const bool edge = base + KT - 1 > w_first || base <= w_last - l.window;
+            const bool edge = base + KT - 1 > w_first || base <= w_last - window;
             float bm[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt)
@@ -360,7 +380,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
                 for (int j = 0; j < 4; ++j) {
                     const int key = base + nt * 8 + 2 * c + (j & 1), p = j < 2 ? pa : pb;
                     float v = s[nt][j] * sl;
-                    if (edge && (key > p || key <= p - l.window)) v = -INFINITY;
+                    if (edge && (key > p || key <= p - window)) v = -INFINITY;
                     s[nt][j] = v;
                     bm[j >> 1] = fmaxf(bm[j >> 1], v);
                 }
@@ -413,8 +433,10 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnArgs a) 
         l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
         const int qi = h ? qb : qa;
         if (qi >= a.S) continue;
-        const float inv = 1.f / l_run[h];
-        __nv_bfloat16 *dst = (__nv_bfloat16 *)a.out + (((size_t)rrow * a.S + qi) * a.H + head) * a.vdim;
+        float inv = 1.f / l_run[h];
+        if constexpr (EXPLICIT)
+            if (a.gate) inv /= 1.f + expf(-__bfloat162float(a.gate[qi * a.gate_stride + head]));
+        __nv_bfloat16 *dst = (__nv_bfloat16 *)a.out + ((size_t)rrow * a.S + qi) * out_stride + (size_t)head * a.vdim;
 #pragma unroll
         for (int i = 0; i < VP / 8; ++i) {
             const int d = i * 8 + 2 * c;
@@ -720,18 +742,18 @@ cudaError_t launch_simt(const WindowAttnArgs &a, dim3 grid, size_t smem, cudaStr
     return launch_kernel(window_attn_kernel<T, REP, 8>, grid, dim3(128), smem, s, a);
 }
 
-template <int DP, int VP>
-cudaError_t launch_mma(const WindowAttnArgs &a, int nrows, cudaStream_t s) {
+template <int DP, int VP, class Args>
+cudaError_t launch_mma(const Args &a, int heads, int nrows, cudaStream_t s) {
     constexpr int smem = 2 * 64 * (DP + VP) * 2;
     static bool configured[64] = {false};
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev >= 0 && dev < 64 && !configured[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(window_attn_mma_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(window_attn_mma_kernel<DP, VP, Args>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return e;
         configured[dev] = true;
     }
-    return launch_kernel(window_attn_mma_kernel<DP, VP>, dim3((a.S + 63) / 64, a.H, nrows), dim3(128), (size_t)smem, s, a);
+    return launch_kernel(window_attn_mma_kernel<DP, VP, Args>, dim3((a.S + 63) / 64, heads, nrows), dim3(128), (size_t)smem, s, a);
 }
 
 template <typename T>
@@ -745,8 +767,8 @@ int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cu
         if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window preparation launch failed: %s", cudaGetErrorString(e));
     }
     if (on_mma && a.S >= 16) {
-        if (a.dim <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, nrows, s) : launch_mma<64, 128>(a, nrows, s);
-        else e = a.vdim <= 64 ? launch_mma<128, 64>(a, nrows, s) : launch_mma<128, 128>(a, nrows, s);
+        if (a.dim <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, a.H, nrows, s) : launch_mma<64, 128>(a, a.H, nrows, s);
+        else e = a.vdim <= 64 ? launch_mma<128, 64>(a, a.H, nrows, s) : launch_mma<128, 128>(a, a.H, nrows, s);
         if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "window attention launch failed: %s", cudaGetErrorString(e));
         return AB2_OK;
     }
@@ -785,6 +807,20 @@ int launch_window(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, cu
 int window_attention(const ab2_kv *kv, WindowAttnArgs a, int nrows, int max_len, ab2_dtype dtype, cudaStream_t s) {
     a.part_acc = kv->part_acc; a.part_ml = kv->part_ml; a.counters = kv->counters;
     return dtype == AB2_F32 ? launch_window<float>(kv, a, nrows, max_len, s) : launch_window<__nv_bfloat16>(kv, a, nrows, max_len, s);
+}
+
+bool prompt_attention_serves(int dim, int tail, int vdim) {
+    return dim % 8 == 0 && tail % 8 == 0 && vdim % 8 == 0 && dim + tail <= 192 && vdim <= 128;
+}
+
+int prompt_attention(const PromptAttnArgs &a, cudaStream_t s) {
+    const int d = a.dim + a.tail_dims;
+    cudaError_t e;
+    if (d <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, a.heads, 1, s) : launch_mma<64, 128>(a, a.heads, 1, s);
+    else if (d <= 128) e = a.vdim <= 64 ? launch_mma<128, 64>(a, a.heads, 1, s) : launch_mma<128, 128>(a, a.heads, 1, s);
+    else e = a.vdim <= 64 ? launch_mma<192, 64>(a, a.heads, 1, s) : launch_mma<192, 128>(a, a.heads, 1, s);
+    if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "prompt attention launch failed: %s", cudaGetErrorString(e));
+    return AB2_OK;
 }
 
 }  // namespace ab2

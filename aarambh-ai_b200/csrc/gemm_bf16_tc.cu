@@ -3,6 +3,7 @@
 //   plain      Y[M][N] = epilogue(X[M][K] . W^T)
 //   MOE_GLU    act[r][ff] = glu(s_r (x_r . Wg_e^T), s_r (x_r . Wu_e^T)),  r a sorted pair of expert e
 //   MOE_DOWN   y[perm[r]][N] = act[r][K] . Wd_e^T
+//   GLU        act[m][ff] = glu(x_m . Wg^T, x_m . Wu^T)
 //
 // As in the other tcgen05 kernels of the library the 128 output channels of a tile are the M
 // dimension of tcgen05.mma and NTOK tokens its N dimension, one persistent CTA per SM:
@@ -51,7 +52,7 @@ struct GbShared {
 };
 
 template <int NTOK, int MODE>
-__host__ __device__ constexpr int gb_stage_bytes() { return (MODE == LIN_MOE_GLU ? 2 : 1) * GB_A_BYTES + NTOK * 128; }
+__host__ __device__ constexpr int gb_stage_bytes() { return (MODE == LIN_MOE_GLU || MODE == LIN_GLU ? 2 : 1) * GB_A_BYTES + NTOK * 128; }
 template <int NTOK, int MODE>
 __host__ __device__ constexpr int gb_stages() {
     return GB_RING_BYTES / gb_stage_bytes<NTOK, MODE>() < GB_MAX_STAGES ? GB_RING_BYTES / gb_stage_bytes<NTOK, MODE>() : GB_MAX_STAGES;
@@ -73,7 +74,7 @@ template <int NTOK, int MODE>
 __global__ void __launch_bounds__(GB_THREADS, 1)
 gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap w2map,
                     const __grid_constant__ CUtensorMap xmap, LinArgs a, int *status) {
-    constexpr bool DUAL = MODE == LIN_MOE_GLU, GROUPED = MODE != LIN_DENSE;
+    constexpr bool DUAL = MODE == LIN_MOE_GLU || MODE == LIN_GLU, GROUPED = MODE == LIN_MOE_GLU || MODE == LIN_MOE_DOWN;
     constexpr int STAGES = gb_stages<NTOK, MODE>(), STAGE_BYTES = gb_stage_bytes<NTOK, MODE>();
     constexpr int ACC_COLS = DUAL ? 2 * NTOK : NTOK;  // tensor-memory columns of one accumulator set
     constexpr uint32_t TMEM_COLS = 2 * ACC_COLS;
@@ -221,12 +222,16 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                 if (MODE == LIN_DENSE) {
                     if (n >= a.N) continue;
                     if (a.epi == LIN_F32) {
-                        float *y = (float *)a.y + (size_t)(row0 + c * CW) * a.N + n;
+                        float *y = (float *)a.y + (row0 + c * CW) * a.ldy + n;
+                        if (a.cap > 0.f) {
+#pragma unroll
+                            for (int j = 0; j < CW; ++j) v[j] = __float_as_uint(softcap_value(__uint_as_float(v[j]), a.cap));
+                        }
 #pragma unroll
                         for (int j = 0; j < CW; ++j)
-                            if (c * CW + j < cnt) y[(size_t)j * a.N] = __uint_as_float(v[j]);
+                            if (c * CW + j < cnt) y[j * a.ldy] = __uint_as_float(v[j]);
                     } else {
-                        __nv_bfloat16 *y = (__nv_bfloat16 *)a.y + (size_t)(row0 + c * CW) * a.N + n;
+                        __nv_bfloat16 *y = (__nv_bfloat16 *)a.y + (row0 + c * CW) * a.ldy + n;
                         const bool act = a.epi == LIN_ACT, silu = n < a.act_n;
 #pragma unroll
                         for (int j = 0; j < CW; ++j) {
@@ -235,14 +240,14 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                                 const float sg = __fdividef(1.f, 1.f + __expf(-f));
                                 f = silu ? f * sg : sg;
                             }
-                            if (c * CW + j < cnt) y[(size_t)j * a.N] = __float2bfloat16_rn(f);
+                            if (c * CW + j < cnt) y[j * a.ldy] = __float2bfloat16_rn(f);
                         }
                     }
                 } else {
                     // lane j holds the pair (and its weight) of the block's token j
                     const int my_row = row0 + c * CW + lane;
-                    const int my_pair = lane < CW && c * CW + lane < cnt ? a.r.perm[my_row] : 0;
-                    const float my_score = DUAL ? a.r.score[my_pair] : 0.f;
+                    const int my_pair = GROUPED && lane < CW && c * CW + lane < cnt ? a.r.perm[my_row] : 0;
+                    const float my_score = MODE == LIN_MOE_GLU && a.scored ? a.r.score[my_pair] : 1.f;
 #pragma unroll
                     for (int j = 0; j < CW; ++j) {
                         const int pair = __shfl_sync(0xffffffffu, my_pair, j);
@@ -250,9 +255,9 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_const
                         if (c * CW + j >= cnt || n >= a.N) continue;
                         if (DUAL)
                             ((__nv_bfloat16 *)a.y)[(size_t)(row0 + c * CW + j) * a.N + n] = __float2bfloat16_rn(
-                                clamped_glu_value(sc * __uint_as_float(v[j]), sc * __uint_as_float(v[16 + j % 16]), a.limit));
+                                glu_value(a.glu, sc * __uint_as_float(v[j]), sc * __uint_as_float(v[16 + j % 16]), a.limit));
                         else
-                            ((float *)a.y)[(size_t)pair * a.N + n] = __uint_as_float(v[j]);
+                            ((float *)a.y)[(size_t)pair * a.N + n] = a.out_scale * __uint_as_float(v[j]);
                     }
                 }
             }
@@ -278,10 +283,11 @@ int launch_tc(const LinArgs &a, cudaStream_t s) {
     int rc = device_status_word(&status);
     if (rc != AB2_OK) return rc;
     CUtensorMap wmap, w2map, xmap;
-    const int wrows = MODE == LIN_DENSE ? a.N : a.N * a.r.E;
+    constexpr bool GROUPED = MODE == LIN_MOE_GLU || MODE == LIN_MOE_DOWN;
+    const int wrows = GROUPED ? a.N * a.r.E : a.N;
     rc = make_x_map(&wmap, a.w, wrows, a.K, 128);
-    if (rc == AB2_OK) rc = make_x_map(&w2map, MODE == LIN_MOE_GLU ? a.w2 : a.w, wrows, a.K, 128);
-    if (rc == AB2_OK) rc = make_x_map(&xmap, a.x, a.M, a.K, NTOK);
+    if (rc == AB2_OK) rc = make_x_map(&w2map, MODE == LIN_MOE_GLU || MODE == LIN_GLU ? a.w2 : a.w, wrows, a.K, 128);
+    if (rc == AB2_OK) rc = make_x_map(&xmap, a.x, a.M, a.K, NTOK, MODE == LIN_DENSE ? a.ldx : a.K);
     if (rc != AB2_OK) return rc;
     const size_t smem = 1024 + (size_t)gb_stages<NTOK, MODE>() * gb_stage_bytes<NTOK, MODE>() + sizeof(GbShared);
     static bool configured[64] = {false};  // the attribute is per device
@@ -293,7 +299,7 @@ int launch_tc(const LinArgs &a, cudaStream_t s) {
         configured[dev] = true;
     }
     // at most this many tiles: every expert may leave one token tile part empty
-    const long long m_tiles = (a.M + NTOK - 1) / NTOK + (MODE == LIN_DENSE ? 0 : std::min(a.r.E, a.r.pairs));
+    const long long m_tiles = (a.M + NTOK - 1) / NTOK + (GROUPED ? std::min(a.r.E, a.r.pairs) : 0);
     const int grid = (int)std::min<long long>(m_tiles * ((a.N + 127) / 128), device_sm_count());
     cudaError_t e = launch_kernel(gemm_bf16_tc_kernel<NTOK, MODE>, dim3(grid), dim3(GB_THREADS), smem, s, wmap, w2map, xmap, a, status);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "bf16 GEMM launch failed: %s", cudaGetErrorString(e));
@@ -307,16 +313,18 @@ int gemm_bf16_tc(const LinArgs &a, int mode, cudaStream_t s) {
     // through L2 - its tokens and the 128 (gate and up: 256) weight rows.  An expert's rows are counted with what
     // routing spreads around their mean.
     const int sms = device_sm_count(), n_tiles = (a.N + 127) / 128;
-    const int groups = mode == LIN_DENSE ? 1 : std::min(a.r.E, a.r.pairs);
-    const double rows = mode == LIN_DENSE ? a.M : (double)a.M / groups + std::sqrt((double)a.M / groups);
+    const bool grouped = mode == LIN_MOE_GLU || mode == LIN_MOE_DOWN, dual = mode == LIN_MOE_GLU || mode == LIN_GLU;
+    const int groups = grouped ? std::min(a.r.E, a.r.pairs) : 1;
+    const double rows = !grouped ? a.M : (double)a.M / groups + std::sqrt((double)a.M / groups);
     auto cost = [&](int ntok) {
         const double tiles = std::ceil(rows / ntok) * n_tiles * groups;
-        return std::ceil(tiles / sms) * (ntok + (mode == LIN_MOE_GLU ? 256 : 128));
+        return std::ceil(tiles / sms) * (ntok + (dual ? 256 : 128));
     };
     if (mode == LIN_DENSE) {
         if (cost(256) <= cost(128) && cost(256) <= cost(64)) return launch_tc<256, LIN_DENSE>(a, s);
         return cost(128) <= cost(64) ? launch_tc<128, LIN_DENSE>(a, s) : launch_tc<64, LIN_DENSE>(a, s);
     }
+    if (mode == LIN_GLU) return cost(128) <= cost(64) ? launch_tc<128, LIN_GLU>(a, s) : launch_tc<64, LIN_GLU>(a, s);
     AB2_REQUIRE(a.r.E <= GB_MAX_EXPERTS, AB2_ERR_UNSUPPORTED, "%d experts exceed the %d the grouped GEMM serves", a.r.E, GB_MAX_EXPERTS);
     if (mode == LIN_MOE_GLU) return cost(128) <= cost(64) ? launch_tc<128, LIN_MOE_GLU>(a, s) : launch_tc<64, LIN_MOE_GLU>(a, s);
     if (cost(256) <= cost(128) && cost(256) <= cost(64)) return launch_tc<256, LIN_MOE_DOWN>(a, s);

@@ -1,12 +1,13 @@
 // Decode linears over dense bf16 weights: HBM-bound streaming on the warp-level tensor cores.
 //
-// A CTA owns 16 weight rows (LIN_MOE_GLU: 8 gate rows and the 8 matching up rows) and its 8 warps
+// A CTA owns 16 weight rows (with a gated unit: 8 gate rows and the 8 matching up rows) and its 8 warps
 // deal out K in chunks of 32 columns.  Per chunk a lane reads 16 bytes of row g, 16 of row g + 8
 // and 16 of each of its tokens (g = lane / 4; lane % 4 picks the 8 columns), which are two
 // mma.sync.m16n8k16 fragments as they stand: the same permutation of K on both operands leaves the
 // dot product alone.  Weights are the rows of the MMA, up to 8 * NT tokens its columns; the warps'
 // sums meet in shared memory.  The first weights are requested before the dependency wait.
-// The grouped modes run one CTA column per active expert and walk that expert's pairs.
+// The grouped modes run one CTA column per active expert and walk that expert's pairs; a batch of
+// weights (one per head) runs one grid layer each.
 #include <algorithm>
 
 #include "linear_bf16.cuh"
@@ -30,6 +31,7 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1
 
 template <int MODE, int NT>
 __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
+    constexpr bool GROUPED = MODE == LIN_MOE_GLU || MODE == LIN_MOE_DOWN, DUAL = MODE == LIN_MOE_GLU || MODE == LIN_GLU;
     constexpr int TOK = 8 * NT;
     __shared__ float red[GV_WARPS][TOK][17];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
@@ -38,7 +40,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
 
     int r0 = 0, cnt = a.M, tile0 = blockIdx.y * TOK, tile_step = gridDim.y * TOK;
     size_t wbase = 0;
-    if (MODE != LIN_DENSE) {
+    if (GROUPED) {
         pdl_wait();
         pdl_launch_dependents();
         if ((int)blockIdx.y >= a.r.active[0]) return;
@@ -48,9 +50,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
         wbase = (size_t)e * a.N * a.K;
         tile0 = 0; tile_step = TOK;
     }
-    const int n0 = blockIdx.x * (MODE == LIN_MOE_GLU ? 8 : 16);
+    if (MODE == LIN_DENSE) wbase = (size_t)blockIdx.z * a.wb;
+    const int n0 = blockIdx.x * (DUAL ? 8 : 16);
     const __nv_bfloat16 *wa = a.w + wbase + (size_t)min(n0 + g, a.N - 1) * a.K + c * 8;
-    const __nv_bfloat16 *wb = MODE == LIN_MOE_GLU ? a.w2 + wbase + (size_t)min(n0 + g, a.N - 1) * a.K + c * 8
+    const __nv_bfloat16 *wb = DUAL ? a.w2 + wbase + (size_t)min(n0 + g, a.N - 1) * a.K + c * 8
                                                   : a.w + wbase + (size_t)min(n0 + g + 8, a.N - 1) * a.K + c * 8;
     uint4 va[GV_UNROLL], vb[GV_UNROLL];
     auto load_w = [&](int ch0) {
@@ -63,11 +66,12 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
         }
     };
     load_w(warp);
-    if (MODE == LIN_DENSE) {
+    if (!GROUPED) {
         pdl_wait();
         pdl_launch_dependents();
     }
-    const __nv_bfloat16 *x = (const __nv_bfloat16 *)a.x;
+    const __nv_bfloat16 *x = (const __nv_bfloat16 *)a.x + (MODE == LIN_DENSE ? blockIdx.z * a.xb : 0);
+    const size_t ldx = MODE == LIN_DENSE ? a.ldx : a.K;
     for (int m0 = tile0; m0 < cnt; m0 += tile_step) {
         const __nv_bfloat16 *xp[NT];
         bool xv[NT];
@@ -77,7 +81,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
             xv[j] = m < cnt;
             const int mm = xv[j] ? m : cnt - 1;
             const int row = MODE == LIN_MOE_GLU ? a.r.perm[r0 + mm] / a.r.top : r0 + mm;
-            xp[j] = x + (size_t)row * a.K + c * 8;
+            xp[j] = x + row * ldx + c * 8;
         }
         float acc[NT][4];
 #pragma unroll
@@ -106,7 +110,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
             red[warp][j * 8 + 2 * c + 1][g + 8] = acc[j][3];
         }
         __syncthreads();
-        constexpr int ROWS = MODE == LIN_MOE_GLU ? 8 : 16;
+        constexpr int ROWS = DUAL ? 8 : 16;
         for (int i = threadIdx.x; i < ROWS * TOK; i += GV_WARPS * 32) {
             const int row = i % ROWS, t = i / ROWS, m = m0 + t, n = n0 + row;
             if (m >= cnt || n >= a.N) continue;
@@ -114,17 +118,21 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
 #pragma unroll
             for (int w = 0; w < GV_WARPS; ++w) {
                 v += red[w][t][row];
-                if (MODE == LIN_MOE_GLU) v2 += red[w][t][row + 8];
+                if (DUAL) v2 += red[w][t][row + 8];
             }
-            if (MODE == LIN_MOE_GLU) {
-                const float s = a.r.score[a.r.perm[r0 + m]];
-                ((__nv_bfloat16 *)a.y)[(size_t)(r0 + m) * a.N + n] = __float2bfloat16_rn(clamped_glu_value(s * v, s * v2, a.limit));
+            if (DUAL) {
+                const float s = MODE == LIN_MOE_GLU && a.scored ? a.r.score[a.r.perm[r0 + m]] : 1.f;
+                ((__nv_bfloat16 *)a.y)[(size_t)(r0 + m) * a.N + n] = __float2bfloat16_rn(glu_value(a.glu, s * v, s * v2, a.limit));
             } else if (MODE == LIN_MOE_DOWN) {
-                ((float *)a.y)[(size_t)a.r.perm[r0 + m] * a.N + n] = v;
+                ((float *)a.y)[(size_t)a.r.perm[r0 + m] * a.N + n] = a.out_scale * v;
             } else {
-                const size_t o = (size_t)m * a.N + n;
-                if (a.epi == LIN_F32) ((float *)a.y)[o] = v;
-                else ((__nv_bfloat16 *)a.y)[o] = __float2bfloat16_rn(a.epi == LIN_ACT ? lin_act_value(v, n < a.act_n) : v);
+                const size_t o = blockIdx.z * a.yb + m * a.ldy + n;
+                if (a.epi == LIN_F32) ((float *)a.y)[o] = softcap_value(v, a.cap);
+                else {
+                    if (a.epi == LIN_ACT) v = lin_act_value(v, n < a.act_n);
+                    if (a.epi == LIN_GATE) v *= lin_act_value(__bfloat162float(((const __nv_bfloat16 *)a.gate)[m * a.gate_ld + blockIdx.z]), false);
+                    ((__nv_bfloat16 *)a.y)[o] = __float2bfloat16_rn(v);
+                }
             }
         }
         __syncthreads();
@@ -133,11 +141,12 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_bf16_kernel(LinArgs a) {
 
 template <int MODE>
 cudaError_t launch_gemv(const LinArgs &a, cudaStream_t s) {
-    const int rows = MODE == LIN_MOE_GLU ? 8 : 16;
+    constexpr bool GROUPED = MODE == LIN_MOE_GLU || MODE == LIN_MOE_DOWN;
+    const int rows = MODE == LIN_MOE_GLU || MODE == LIN_GLU ? 8 : 16;
     // most pairs one expert can get: every token once
-    const int m = MODE == LIN_DENSE ? a.M : a.r.pairs / a.r.top;
+    const int m = GROUPED ? a.r.pairs / a.r.top : a.M;
     const int nt = m <= 8 ? 1 : m <= 16 ? 2 : 4;
-    dim3 grid((a.N + rows - 1) / rows, MODE == LIN_DENSE ? (m + 8 * nt - 1) / (8 * nt) : std::min(a.r.E, a.r.pairs));
+    dim3 grid((a.N + rows - 1) / rows, GROUPED ? std::min(a.r.E, a.r.pairs) : (m + 8 * nt - 1) / (8 * nt), MODE == LIN_DENSE ? a.batch : 1);
     if (nt == 1) return launch_kernel(gemv_bf16_kernel<MODE, 1>, grid, dim3(GV_WARPS * 32), 0, s, a);
     if (nt == 2) return launch_kernel(gemv_bf16_kernel<MODE, 2>, grid, dim3(GV_WARPS * 32), 0, s, a);
     return launch_kernel(gemv_bf16_kernel<MODE, 4>, grid, dim3(GV_WARPS * 32), 0, s, a);
@@ -148,6 +157,7 @@ cudaError_t launch_gemv(const LinArgs &a, cudaStream_t s) {
 int gemv_bf16(const LinArgs &a, int mode, cudaStream_t s) {
     cudaError_t e = mode == LIN_DENSE     ? launch_gemv<LIN_DENSE>(a, s)
                     : mode == LIN_MOE_GLU ? launch_gemv<LIN_MOE_GLU>(a, s)
+                    : mode == LIN_GLU     ? launch_gemv<LIN_GLU>(a, s)
                                           : launch_gemv<LIN_MOE_DOWN>(a, s);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "bf16 GEMV launch failed: %s", cudaGetErrorString(e));
     return AB2_OK;

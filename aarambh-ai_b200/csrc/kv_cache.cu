@@ -14,6 +14,7 @@
 #include "common.cuh"
 #include "kv_cache.cuh"
 #include "ops.cuh"
+#include "stack.cuh"
 
 using namespace ab2;
 
@@ -255,7 +256,7 @@ AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n
     for (int i = 0; i < batch; ++i) kv->saved_len[i] = -1;
     const int esz = (int)kv_elem_size(dtype);
     kv->max_splits = AB2_KV_MAX_SPLITS;
-    size_t part = 0, heads = 0;  // an attention layer has at most `heads` (KV head, head group) pairs
+    size_t part = 0, heads = 0, latent_part = 0;  // an attention layer has at most `heads` (KV head, head group) pairs
     cudaError_t e = cudaSuccess;
     for (int i = 0; i < n_layers && e == cudaSuccess; ++i) {
         const ab2_layer_spec &sp = specs[i];
@@ -268,16 +269,22 @@ AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n
             if (e == cudaSuccess) e = cudaMemset(l.state, 0, (size_t)batch * layer_state_elems(l) * 4);
             continue;
         }
-        l.kvh = sp.kv_heads;
+        if (sp.mixer == AB2_MIX_LATENT) {  // one row per token: the latent, then the shared key part
+            l.kvh = 1; l.kd = sp.kv_rank + sp.rot_dims; l.vd = 0;
+            latent_part = std::max(latent_part, latent_part_bytes(sp));
+        } else {
+            l.kvh = sp.kv_heads;
+        }
         l.kds = (l.kd + 7) / 8 * 8; l.vds = (l.vd + 7) / 8 * 8;
         // a step of max_step tokens is appended before its queries look back a whole window
         l.window = sp.window > 0 ? std::min(sp.window, capacity) : capacity;
         l.cap = (int)std::min<long long>(capacity, (long long)l.window - 1 + max_step);
-        for (int which = 0; which < 2 && e == cudaSuccess; ++which) {
+        for (int which = 0; which < (l.vd > 0 ? 2 : 1) && e == cudaSuccess; ++which) {
             void **p = which ? &l.v : &l.k;
             e = cudaMalloc(p, (size_t)batch * layer_row_bytes(l, which, esz));
             if (e == cudaSuccess) e = cudaMemset(*p, 0, (size_t)batch * layer_row_bytes(l, which, esz));
         }
+        if (l.vd == 0) continue;
         part = std::max(part, (size_t)sp.heads * l.vd);
         heads = std::max(heads, (size_t)sp.heads);
     }
@@ -286,10 +293,10 @@ AB2_API int ab2_kv_create_stack(ab2_kv **out, const ab2_layer_spec *specs, int n
     if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->lens_host, (size_t)batch * 4);
     if (e == cudaSuccess) e = cudaMalloc((void **)&kv->rows_dev, (size_t)batch * 4);
     if (e == cudaSuccess) e = cudaMallocHost((void **)&kv->rows_host, (size_t)batch * 4);
-    kv->part_acc_bytes = (size_t)batch * kv->max_splits * part * 4;
-    kv->part_ml_bytes = (size_t)batch * kv->max_splits * heads * 2 * 4;
-    if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_acc, kv->part_acc_bytes);
-    if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->part_ml, kv->part_ml_bytes);
+    kv->part_acc_bytes = std::max((size_t)batch * kv->max_splits * part * 4, latent_part);
+    kv->part_ml_bytes = std::max((size_t)batch * kv->max_splits * heads * 2 * 4, latent_part > 0 ? latent_part_ml_bytes() : 0);
+    if (e == cudaSuccess && kv->part_acc_bytes > 0) e = cudaMalloc((void **)&kv->part_acc, kv->part_acc_bytes);
+    if (e == cudaSuccess && kv->part_ml_bytes > 0) e = cudaMalloc((void **)&kv->part_ml, kv->part_ml_bytes);
     kv->counter_bytes = (size_t)batch * heads * 4;
     if (e == cudaSuccess && part > 0) e = cudaMalloc((void **)&kv->counters, kv->counter_bytes);
     if (e == cudaSuccess && part > 0) e = cudaMemset(kv->counters, 0, kv->counter_bytes);
@@ -469,7 +476,7 @@ static int clone_stack(ab2_kv **out, const ab2_kv *src, cudaStream_t s) {
         if (a.recurrent) {
             dup((void **)&b.state, a.state, (size_t)src->B * layer_state_elems(a) * 4, true);
         } else {
-            dup(&b.k, a.k, (size_t)src->B * layer_row_bytes(a, false, esz), true);
+            dup(&b.k, a.k, (size_t)src->B * layer_row_bytes(a, false, esz), true);  // a latent layer has no values of its own
             dup(&b.v, a.v, (size_t)src->B * layer_row_bytes(a, true, esz), true);
         }
     }

@@ -6,7 +6,8 @@
 #define AB2_KV_MAX_SPLITS 64
 
 // What one layer of a layer stack keeps per sequence: either the last `cap` keys and values
-// (position p in slot p % cap), or a recurrent state.
+// (position p in slot p % cap), or a recurrent state.  A latent layer keeps one row per token (kvh 1,
+// vd 0): the latent and the key part that its heads share.
 struct KvLayer {
     bool recurrent;
     int kvh, kd, vd;      // attention: heads, key and value size; recurrent: heads and the two state dimensions

@@ -342,7 +342,8 @@ static int check_forward(ab2_model *m, ab2_kv *kv, const void *ids, int S, int r
     AB2_REQUIRE(m && kv && ids, AB2_ERR_BAD_ARG, "null argument");
     AB2_REQUIRE(m->finalized, AB2_ERR_BAD_ARG, "model is not finalised");
     const ab2_model_config &c = m->cfg;
-    AB2_REQUIRE(kv->L == c.n_layers, AB2_ERR_BAD_SHAPE, "expected %d cache layers, got %d", c.n_layers, kv->L);
+    const int cache_layers = m->stack ? stack_runs(m->stack) : c.n_layers;
+    AB2_REQUIRE(kv->L == cache_layers, AB2_ERR_BAD_SHAPE, "expected %d cache layers, got %d", cache_layers, kv->L);
     if (m->stack) {
         int rc = stack_check_cache(m->stack, kv, S);
         if (rc != AB2_OK) return rc;
@@ -408,6 +409,27 @@ AB2_API int ab2_model_create_stack(ab2_model **out, const ab2_model_config *cfg,
     m->stack = st; m->cfg = *cfg; m->dtype = dtype; m->max_tokens = max_tokens;
     *out = m;
     return AB2_OK;
+}
+
+AB2_API int ab2_model_set_form(ab2_model *m, const ab2_stack_form *form) {
+    AB2_REQUIRE(m && form, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(m->stack, AB2_ERR_UNSUPPORTED, "the dense decoder has one form");
+    m->finalized = false;
+    return stack_set_form(m->stack, *form);
+}
+
+AB2_API int ab2_model_set_loop_steps(ab2_model *m, const float *steps) {
+    AB2_REQUIRE(m && steps, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(m->stack, AB2_ERR_UNSUPPORTED, "the dense decoder has no loop");
+    m->finalized = false;
+    return stack_set_loop_steps(m->stack, steps);
+}
+
+AB2_API int ab2_model_set_expert_table(ab2_model *m, int layer, const int *table) {
+    AB2_REQUIRE(m && table, AB2_ERR_BAD_ARG, "null argument");
+    AB2_REQUIRE(m->stack, AB2_ERR_UNSUPPORTED, "the dense decoder has no experts");
+    m->finalized = false;
+    return stack_set_expert_table(m->stack, layer, table);
 }
 
 AB2_API int ab2_model_destroy(ab2_model *m) {

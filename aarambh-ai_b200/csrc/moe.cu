@@ -1,5 +1,6 @@
-// Routing of a mixture of experts: sigmoid scores of the router's f32 logits, the `top` largest per
-// token, and the (token, expert) pairs sorted by expert for the grouped linears.
+// Routing of a mixture of experts: sigmoid scores of the router's f32 logits and the `top` largest per
+// token, or experts named by a table of token ids; and the (token, expert) pairs sorted by expert for the
+// grouped linears.
 #include <algorithm>
 #include <climits>
 
@@ -46,17 +47,10 @@ __global__ void __launch_bounds__(256) moe_choose_kernel(const float *logits, in
     if (t < T) choose_experts(logits + (size_t)t * r.E, r.E, r.top, r.expert + (size_t)t * r.top, r.score + (size_t)t * r.top, threadIdx.x & 31);
 }
 
-// One CTA: (with CHOOSE) the choice, then counting sort of the pairs by expert.
-template <bool CHOOSE>
-__global__ void __launch_bounds__(1024) moe_sort_kernel(const float *logits, int T, MoeRoute r) {
-    __shared__ int count[MAX_EXPERTS], next[MAX_EXPERTS];
-    pdl_wait();
-    pdl_launch_dependents();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+// Counting sort of the pairs by expert, by one CTA whose threads have written r.expert.
+__device__ __forceinline__ void sort_pairs(const MoeRoute &r, int *count, int *next) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int e = threadIdx.x; e < r.E; e += blockDim.x) count[e] = 0;
-    if (CHOOSE)
-        for (int t = warp; t < T; t += nw)
-            choose_experts(logits + (size_t)t * r.E, r.E, r.top, r.expert + (size_t)t * r.top, r.score + (size_t)t * r.top, lane);
     __syncthreads();
     for (int p = threadIdx.x; p < r.pairs; p += blockDim.x) atomicAdd(&count[r.expert[p]], 1);
     __syncthreads();
@@ -82,6 +76,34 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const float *logits, int
     for (int p = threadIdx.x; p < r.pairs; p += blockDim.x) r.perm[atomicAdd(&next[r.expert[p]], 1)] = p;
 }
 
+// One CTA: (with CHOOSE) the choice, then the sort.
+template <bool CHOOSE>
+__global__ void __launch_bounds__(1024) moe_sort_kernel(const float *logits, int T, MoeRoute r) {
+    __shared__ int count[MAX_EXPERTS], next[MAX_EXPERTS];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+    if (CHOOSE)
+        for (int t = warp; t < T; t += nw)
+            choose_experts(logits + (size_t)t * r.E, r.E, r.top, r.expert + (size_t)t * r.top, r.score + (size_t)t * r.top, lane);
+    sort_pairs(r, count, next);
+}
+
+// One CTA per layer whose experts are named by the token id.
+__global__ void __launch_bounds__(1024) moe_table_kernel(const MoeTable *tables, const uint32_t *ids, int vocab, int T) {
+    __shared__ int count[MAX_EXPERTS], next[MAX_EXPERTS];
+    pdl_wait();
+    pdl_launch_dependents();
+    const MoeTable m = tables[blockIdx.x];
+    MoeRoute r = m.r;
+    r.pairs = T * r.top;
+    for (int p = threadIdx.x; p < r.pairs; p += blockDim.x) {
+        const uint32_t id = min(ids[p / r.top], (uint32_t)vocab - 1u);  // ids are validated on the host; keep reads in range
+        r.expert[p] = m.table[(size_t)id * r.top + p % r.top];
+    }
+    sort_pairs(r, count, next);
+}
+
 }  // namespace
 
 int moe_route(const float *logits, int T, const MoeRoute &r, cudaStream_t s) {
@@ -93,6 +115,12 @@ int moe_route(const float *logits, int T, const MoeRoute &r, cudaStream_t s) {
         e = launch_kernel(moe_choose_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, T, r);
         if (e == cudaSuccess) e = launch_kernel(moe_sort_kernel<false>, dim3(1), dim3(1024), 0, s, logits, T, r);
     }
+    if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "routing launch failed: %s", cudaGetErrorString(e));
+    return AB2_OK;
+}
+
+int moe_route_tables(const MoeTable *tables_dev, int n, const uint32_t *ids, int vocab, int T, cudaStream_t s) {
+    cudaError_t e = launch_kernel(moe_table_kernel, dim3(n), dim3(T <= 8 ? 128 : 1024), 0, s, tables_dev, ids, vocab, T);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "routing launch failed: %s", cudaGetErrorString(e));
     return AB2_OK;
 }

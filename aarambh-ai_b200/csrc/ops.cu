@@ -252,10 +252,186 @@ __global__ void residual_norm_kernel(ResidualNormArgs a) {
     }
 }
 
+// RN_EMBED and RN_ADD with what a stack may ask for besides (see ResidualNormArgs):
+//   RN_EMBED   x = embedding, normed where w is given (kept in x0), plus the vector `add`
+//   RN_ADD     x += norm of the summed parts, then plus x0 and the vector `add` where given
+// and in both cases out = RMSNorm(x; w_next), or x itself without w_next.
+template <typename T, int MODE>
+__global__ void residual_step_kernel(ResidualNormArgs a) {
+    extern __shared__ float vrow[];
+    __shared__ float warp_sums[2][32];
+    const size_t t = blockIdx.x;
+    const int nw = blockDim.x >> 5;
+    pdl_wait();
+    pdl_launch_dependents();
+    uint32_t id = 0;
+    if (MODE == RN_EMBED) {
+        id = a.ids[t];
+        if (id >= (uint32_t)a.vocab) id = a.vocab - 1;  // ids are validated on the host; keep reads in range
+    }
+    const float *parts = a.parts + t * (size_t)a.nparts * a.d;
+    float *x = a.x + t * (size_t)a.d;
+    auto block_sum = [&](float v, int which) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        if ((threadIdx.x & 31) == 0) warp_sums[which][threadIdx.x >> 5] = v;
+        __syncthreads();
+        v = 0.f;
+        for (int w = 0; w < nw; ++w) v += warp_sums[which][w];
+        return v;
+    };
+    struct alignas(4 * sizeof(T)) Quad { T e[4]; };
+    const bool vec = (a.d & 3) == 0;
+    const int n = vec ? a.d / 4 : a.d;  // float4 or single values; a thread reads back only what it wrote
+    float4 *v4 = reinterpret_cast<float4 *>(vrow);
+    float sum = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        if (vec) {
+            float4 v;
+            if (MODE == RN_EMBED) {
+                const uint2 e = reinterpret_cast<const uint2 *>(a.table + (size_t)id * a.d)[i];
+                v = make_float4(__uint_as_float(e.x << 16), __uint_as_float(e.x & 0xffff0000u), __uint_as_float(e.y << 16),
+                                __uint_as_float(e.y & 0xffff0000u));
+            } else {
+                v = reinterpret_cast<const float4 *>(parts)[i];
+                for (int p = 1; p <= a.nparts; ++p) {
+                    if (p == a.nparts && !a.extra) break;
+                    const float4 q = reinterpret_cast<const float4 *>(p < a.nparts ? parts + (size_t)p * a.d : a.extra + t * (size_t)a.d)[i];
+                    v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+                }
+            }
+            v4[i] = v;
+            sum = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sum))));
+        } else {
+            float v;
+            if (MODE == RN_EMBED) {
+                v = __bfloat162float(a.table[(size_t)id * a.d + i]);
+            } else {
+                v = parts[i];
+                for (int p = 1; p < a.nparts; ++p) v += parts[(size_t)p * a.d + i];
+                if (a.extra) v += a.extra[t * (size_t)a.d + i];
+            }
+            vrow[i] = v;
+            sum = fmaf(v, v, sum);
+        }
+    }
+    const float inv = MODE == RN_ADD || a.w ? 1.f / sqrtf(block_sum(sum, 0) / (float)a.d + a.eps) : 1.f;
+    sum = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const int lanes = vec ? 4 : 1;
+        float v[4], ad[4] = {0.f, 0.f, 0.f, 0.f}, x0[4] = {0.f, 0.f, 0.f, 0.f};
+        if (vec) {
+            const float4 r = v4[i], w = a.w ? reinterpret_cast<const float4 *>(a.w)[i] : make_float4(1.f, 1.f, 1.f, 1.f);
+            v[0] = r.x * inv * w.x; v[1] = r.y * inv * w.y; v[2] = r.z * inv * w.z; v[3] = r.w * inv * w.w;
+            if (MODE == RN_ADD) {
+                const float4 q = reinterpret_cast<const float4 *>(x)[i];
+                v[0] += q.x; v[1] += q.y; v[2] += q.z; v[3] += q.w;
+                if (a.x0) *reinterpret_cast<float4 *>(x0) = reinterpret_cast<const float4 *>(a.x0 + t * (size_t)a.d)[i];
+            } else if (a.x0) {
+                reinterpret_cast<float4 *>(a.x0 + t * (size_t)a.d)[i] = make_float4(v[0], v[1], v[2], v[3]);
+            }
+            if (a.add) *reinterpret_cast<float4 *>(ad) = reinterpret_cast<const float4 *>(a.add)[i];
+        } else {
+            v[0] = vrow[i] * inv * (a.w ? a.w[i] : 1.f);
+            if (MODE == RN_ADD) {
+                v[0] += x[i];
+                if (a.x0) x0[0] = a.x0[t * (size_t)a.d + i];
+            } else if (a.x0) {
+                a.x0[t * (size_t)a.d + i] = v[0];
+            }
+            if (a.add) ad[0] = a.add[i];
+        }
+        for (int j = 0; j < lanes; ++j) {
+            v[j] = v[j] + x0[j] + ad[j];
+            sum = fmaf(v[j], v[j], sum);
+        }
+        if (vec) {
+            const float4 r = make_float4(v[0], v[1], v[2], v[3]);
+            reinterpret_cast<float4 *>(x)[i] = r;
+            v4[i] = r;
+        } else {
+            x[i] = vrow[i] = v[0];
+        }
+    }
+    if (a.out == nullptr) return;
+    const float inv2 = a.w_next ? 1.f / sqrtf(block_sum(sum, 1) / (float)a.d + a.eps) : 1.f;
+    T *out = (T *)a.out + t * (size_t)a.d;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        if (vec) {
+            const float4 r = v4[i], w = a.w_next ? reinterpret_cast<const float4 *>(a.w_next)[i] : make_float4(1.f, 1.f, 1.f, 1.f);
+            Quad q;
+            q.e[0] = from_f32<T>(r.x * inv2 * w.x); q.e[1] = from_f32<T>(r.y * inv2 * w.y);
+            q.e[2] = from_f32<T>(r.z * inv2 * w.z); q.e[3] = from_f32<T>(r.w * inv2 * w.w);
+            reinterpret_cast<Quad *>(out)[i] = q;
+        } else {
+            out[i] = from_f32<T>(vrow[i] * inv2 * (a.w_next ? a.w_next[i] : 1.f));
+        }
+    }
+}
+
+// out = a N(z) + b N(z^2) + c N(z^3) + e over rows of n values, N the division by the root mean square
+// of the row (see PolyNorm in stack.cuh).  One CTA per token.
+template <typename T, int V>
+__global__ void poly_norm_kernel(PolyNormArgs p) {
+    __shared__ float sums[3][32];
+    pdl_wait();
+    pdl_launch_dependents();
+    const T *z = (const T *)p.z + (size_t)blockIdx.x * p.n;
+    T *out = (T *)p.out + (size_t)blockIdx.x * p.n;
+    struct alignas(V * sizeof(T)) Vec { T e[V]; };
+    float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+    for (int i = threadIdx.x; i < p.n / V; i += blockDim.x) {
+        const Vec q = reinterpret_cast<const Vec *>(z)[i];
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+            const float v = to_f32(q.e[j]), w = v * v;
+            s2 += w;
+            s4 = fmaf(w, w, s4);
+            s6 = fmaf(w * w, w, s6);
+        }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        s2 += __shfl_xor_sync(0xffffffffu, s2, o);
+        s4 += __shfl_xor_sync(0xffffffffu, s4, o);
+        s6 += __shfl_xor_sync(0xffffffffu, s6, o);
+    }
+    const int w = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) == 0) { sums[0][w] = s2; sums[1][w] = s4; sums[2][w] = s6; }
+    __syncthreads();
+    s2 = s4 = s6 = 0.f;
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) { s2 += sums[0][i]; s4 += sums[1][i]; s6 += sums[2][i]; }
+    const float n = (float)p.n;
+    const float a = p.a / sqrtf(s2 / n + p.eps), b = p.b / sqrtf(s4 / n + p.eps), c = p.c / sqrtf(s6 / n + p.eps);
+    for (int i = threadIdx.x; i < p.n / V; i += blockDim.x) {
+        const Vec q = reinterpret_cast<const Vec *>(z)[i];
+        Vec r;
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+            const float v = to_f32(q.e[j]);
+            r.e[j] = from_f32<T>(fmaf(v, fmaf(v, fmaf(v, c, b), a), p.e));
+        }
+        reinterpret_cast<Vec *>(out)[i] = r;
+    }
+}
+
+int launch_poly_norm(const PolyNormArgs &p, int rows, ab2_dtype dtype, cudaStream_t s) {
+    const bool vec = p.n % 8 == 0;
+    const int threads = std::min(1024, std::max(128, (p.n / 16 + 31) / 32 * 32));
+    cudaError_t e;
+    if (dtype == AB2_F32) e = vec ? launch_kernel(poly_norm_kernel<float, 4>, dim3(rows), dim3(threads), 0, s, p) : launch_kernel(poly_norm_kernel<float, 1>, dim3(rows), dim3(threads), 0, s, p);
+    else e = vec ? launch_kernel(poly_norm_kernel<__nv_bfloat16, 8>, dim3(rows), dim3(threads), 0, s, p) : launch_kernel(poly_norm_kernel<__nv_bfloat16, 1>, dim3(rows), dim3(threads), 0, s, p);
+    if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "activation launch failed: %s", cudaGetErrorString(e));
+    return AB2_OK;
+}
+
 template <typename T>
 static cudaError_t launch_residual(const ResidualNormArgs &a, int mode, int rows, cudaStream_t s) {
     const int threads = std::min(1024, std::max(128, (a.d / 8 + 31) / 32 * 32));
     const size_t smem = (size_t)a.d * 4;
+    const bool more = a.w_next || a.extra || a.x0 || a.add;
+    if (mode == RN_EMBED && (more || !a.w)) return launch_kernel(residual_step_kernel<T, RN_EMBED>, dim3(rows), dim3(threads), smem, s, a);
+    if (mode == RN_ADD && more) return launch_kernel(residual_step_kernel<T, RN_ADD>, dim3(rows), dim3(threads), smem, s, a);
     switch (mode) {
     case RN_EMBED: return launch_kernel(residual_norm_kernel<T, RN_EMBED>, dim3(rows), dim3(threads), smem, s, a);
     case RN_ADD: return launch_kernel(residual_norm_kernel<T, RN_ADD>, dim3(rows), dim3(threads), smem, s, a);

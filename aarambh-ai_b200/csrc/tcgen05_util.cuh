@@ -108,7 +108,8 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t
                                   const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-inline int make_x_map(CUtensorMap *map, const void *x, int M, int K, int ntok) {
+// Tensor map of a [M][K] bf16 matrix whose rows lie `ld` elements apart (0: K), read in boxes of 64 x ntok.
+inline int make_x_map(CUtensorMap *map, const void *x, int M, int K, int ntok, long long ld = 0) {
     static EncodeTiledFn encode = nullptr;
     if (!encode) {
         void *fn = nullptr;
@@ -118,7 +119,7 @@ inline int make_x_map(CUtensorMap *map, const void *x, int M, int K, int ntok) {
         encode = (EncodeTiledFn)fn;
     }
     cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)M};
-    cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+    cuuint64_t strides[1] = {(cuuint64_t)(ld > 0 ? ld : K) * 2};
     cuuint32_t box[2] = {64, (cuuint32_t)ntok};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(x), dims, strides, box, estr,

@@ -176,12 +176,41 @@ def lightning_attention(cache, cfg, layer: int, qkv: torch.Tensor, powers: torch
     return out
 
 
+def latent_attention(cache, cfg, layer: int, proj: torch.Tensor, norm: torch.Tensor, ukv, tables, eps: float, row0: int = 0,
+                     workspace: torch.Tensor | None = None) -> torch.Tensor:
+    """proj [rows, S, stride] (overwritten): heads (dim + rot_dims) queries | latent | shared key part | gates;
+    ``ukv`` the keys' and values' up projection (``QuantLinear``) -> [rows, S, heads vdim]."""
+    proj = _cuda(proj, "proj")
+    specs, _keep = cfg.c_specs(cfg.runs())
+    sp = specs[layer]
+    rows, S, stride = proj.shape
+    if workspace is None:
+        n = C.c_size_t()
+        check(lib.ab2_latent_workspace(C.byref(sp), rows * S, cache.cap, dtype_code(proj.dtype), C.byref(n)))
+        workspace = torch.empty(n.value, dtype=torch.uint8, device=proj.device)
+    out = torch.empty((rows, S, sp.heads * sp.vdim), dtype=proj.dtype, device=proj.device)
+    cos, sin = tables if tables is not None else (None, None)
+    check(lib.ab2_latent_attention(cache._h, layer, C.byref(sp), proj.data_ptr(), stride, norm.data_ptr(), ukv._h,
+                                   cos.data_ptr() if cos is not None else None, sin.data_ptr() if sin is not None else None, float(eps),
+                                   out.data_ptr(), workspace.data_ptr(), workspace.numel(), S, row0, rows, dtype_code(proj.dtype), stream_ptr()))
+    return out
+
+
+def poly_norm(z: torch.Tensor, coef, eps: float) -> torch.Tensor:
+    """a N(z) + b N(z^2) + c N(z^3) + e over the last dimension, N the division by the root mean square."""
+    z = _cuda(z, "z")
+    out = torch.empty_like(z)
+    check(lib.ab2_poly_norm(z.data_ptr(), out.data_ptr(), z.numel() // z.shape[-1], z.shape[-1], (C.c_float * 4)(*coef), float(eps),
+                            dtype_code(z.dtype), stream_ptr()))
+    return out
+
+
 class MoeExperts:
-    """The feed-forward of ``model.MoeFfn`` over dense bf16 weights: x [tokens, width] -> the chosen
+    """The feed-forward of a ``model.MoeFfn`` with a router over dense bf16 weights: x [tokens, width] -> the chosen
     experts' outputs [tokens, top, width] (f32; their sum is the layer's output)."""
 
     def __init__(self, ffn, router, gate, up, down):
-        self.spec = _lib.LayerSpec(ffn=_lib.FFN_MOE, experts=ffn.experts, top=ffn.top, ff=ffn.ff, limit=ffn.limit)
+        self.spec = _lib.LayerSpec(ffn=_lib.FFN_MOE, experts=ffn.experts, top=ffn.top, ff=ffn.ff, limit=ffn.limit, glu=_lib.GLU[ffn.glu])
         self.router, self.gate, self.up, self.down = router, gate, up, down
         self._work = None
 

@@ -37,11 +37,13 @@ class KVCache:
 
     @classmethod
     def for_stack(cls, cfg, capacity: int, batch: int, max_step: int, dtype: str):
-        """The cache of a layer stack (``StackConfig``): windows in rings, recurrent states beside them."""
-        specs, _keep = cfg.c_specs()
+        """The cache of a layer stack (``StackConfig``): windows in rings, latents, recurrent states beside them;
+        one cache layer for every run of a layer."""
+        order = cfg.runs()
+        specs, _keep = cfg.c_specs(order)
         h = C.c_void_p()
-        check(lib.ab2_kv_create_stack(C.byref(h), specs, len(cfg.layers), batch, capacity, max_step, _KV_DTYPES[dtype]))
-        return cls(capacity, 0, 0, 0, batch, len(cfg.layers), dtype, _handle=h.value)
+        check(lib.ab2_kv_create_stack(C.byref(h), specs, len(order), batch, capacity, max_step, _KV_DTYPES[dtype]))
+        return cls(capacity, 0, 0, 0, batch, len(order), dtype, _handle=h.value)
 
     def update(self, k: torch.Tensor, v: torch.Tensor, row0: int = 0):
         """Appends k, v [rows, S, kv_heads, head_dim] and returns the cached tensors

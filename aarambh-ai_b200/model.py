@@ -219,12 +219,38 @@ class LightningMixer:
 
 
 @dataclass
+class LatentMixer:
+    """Causal softmax attention whose keys and values are projections of one cached latent per token, plus
+    a rotated key part that the heads share."""
+    heads: int
+    dim: int                      # unrotated dimensions of a query and key
+    rot_dims: int                 # rotated ones besides, in adjacent pairs
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float = 10000.0
+    head_gate: bool = False       # a head's output times the sigmoid of a gate value of its own
+
+
+@dataclass
 class MoeFfn:
-    """Mixture of experts: sigmoid scores that multiply the chosen experts' inputs, clamped gated unit."""
+    """Mixture of experts over gated units: ``clamped`` (with ``limit``) or ``silu``.  ``sigmoid`` routing: a
+    router's largest scores, which multiply what the experts read.  ``table`` routing: the token id
+    names the experts, each output weighs 1 / top."""
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = 0.0
+    glu: str = "clamped"
+    routing: str = "sigmoid"
+    shared_ff: int = 0            # width of an expert that runs for every token, 0: none
+
+
+@dataclass
+class PolyFfn:
+    """W_down act(W_up x) with act(z) = a N(z) + b N(z^2) + c N(z^3) + e, N(z) = z / rms(z) over the row."""
+    ff: int
+    coef: tuple                   # a, b, c, e
 
 
 @dataclass
@@ -236,14 +262,29 @@ class StackConfig:
     max_seq_len: int
     rms_norm_eps: float = 1e-5
     tie_embeddings: bool = True
+    embed_norm: bool = True       # the embedding is normed
+    pre_norms: bool = False       # sublayers read a norm of the residual stream
+    loop: tuple | None = None     # (start, stop, times): those layers run that often in a row
+    logit_softcap: float = 0.0    # cap of tanh-capped logits, 0: none
 
-    def c_specs(self):
-        """The layers as an array of ab2_layer_spec (and what it points to)."""
-        arr = (_lib.LayerSpec * len(self.layers))()
+    def runs(self) -> list:
+        """Layer indices in the order in which a pass runs them; each run has a cache layer of its own."""
+        start, stop, times = self.loop or (0, 0, 0)
+        n = len(self.layers)
+        return list(range(start)) + list(range(start, stop)) * times + list(range(stop, n))
+
+    def c_specs(self, order=None):
+        """The layers (or those of ``order``) as an array of ab2_layer_spec (and what it points to)."""
+        order = range(len(self.layers)) if order is None else order
+        arr = (_lib.LayerSpec * len(order))()
         keep = []
-        for s, (mix, ffn) in zip(arr, self.layers):
+        for s, i in zip(arr, order):
+            mix, ffn = self.layers[i]
             s.heads, s.dim, s.vdim = mix.heads, mix.dim, mix.vdim
-            if isinstance(mix, LightningMixer):
+            if isinstance(mix, LatentMixer):
+                s.mixer = _lib.MIX_LATENT
+                s.kv_rank, s.rot_dims, s.rot_base, s.scale, s.head_gate = mix.kv_rank, mix.rot_dims, mix.rot_base, mix.scale, int(mix.head_gate)
+            elif isinstance(mix, LightningMixer):
                 if len(mix.decay) != mix.heads:
                     raise _lib.Ab2Error(-1, f"{len(mix.decay)} decays for {mix.heads} heads")
                 s.mixer = _lib.MIX_LIGHTNING
@@ -254,9 +295,17 @@ class StackConfig:
                 s.kv_heads, s.window, s.scale = mix.kv_heads, mix.window, mix.scale
                 s.rot_dims, s.rot_base, s.qk_norm = mix.rot_dims, mix.rot_base, int(mix.qk_norm)
                 s.v_mix, s.v_lambda = int(mix.v_mix), mix.v_lambda
-            if ffn is not None:
+            if isinstance(ffn, PolyFfn):
+                s.ffn, s.ff = _lib.FFN_POLY, ffn.ff
+                s.poly[:] = ffn.coef
+            elif ffn is not None:
                 s.ffn, s.experts, s.top, s.ff, s.limit = _lib.FFN_MOE, ffn.experts, ffn.top, ffn.ff, ffn.limit
+                s.glu, s.routing, s.shared_ff = _lib.GLU[ffn.glu], _lib.ROUTING[ffn.routing], ffn.shared_ff
         return arr, keep
+
+    def c_form(self):
+        start, stop, times = self.loop or (0, 0, 0)
+        return _lib.StackForm(int(self.embed_norm), int(self.pre_norms), start, stop, times, self.logit_softcap)
 
 
 class StackModel(DecoderModel):
@@ -264,12 +313,16 @@ class StackModel(DecoderModel):
 
     weights: name -> ``QuantLinear.from_bf16`` for ``embedding``, optional ``lm_head`` and
     ``layers.{i}.{in,out}`` (the mixer's input projections as one weight: q | k | v, lightning
-    q | k | v | g) and ``layers.{i}.{gate,up,down,router}`` (the experts one after the other);
-    name -> f32 tensor for ``embed_norm``, ``final_norm``, ``layers.{i}.{norm1,norm2}`` and, in
-    lightning layers, ``layers.{i}.mix_norm``.  Logits are f32."""
+    q | k | v | g, latent q | latent | key part | g and zero rows up to a multiple of 8), latent
+    ``layers.{i}.ukv`` (head by head the rows of its keys and its values), ``layers.{i}.{gate,up,down,router}``
+    (the experts one after the other) and ``layers.{i}.shared_{gate,up,down}``;
+    name -> f32 tensor for ``embed_norm``, ``final_norm``, ``layers.{i}.{norm1,norm2}`` (after the mixer and the
+    feed-forward), with ``pre_norms`` ``layers.{i}.{pre1,pre2}`` (before them), in lightning and latent layers
+    ``layers.{i}.mix_norm``, with a loop ``loop_steps`` [times, d_model]; ``layers.{i}.table`` [vocab, top] int32 where
+    the token id names the experts.  Logits are f32."""
 
-    LINEARS = {"in": 0, "out": 3, "gate": 4, "up": 5, "down": 6, "router": 7}
-    NORMS = {"norm1": 0, "norm2": 1, "mix_norm": 2}
+    LINEARS = {"in": 0, "ukv": 1, "out": 3, "gate": 4, "up": 5, "down": 6, "router": 7, "shared_gate": 8, "shared_up": 9, "shared_down": 10}
+    NORMS = {"norm1": 0, "norm2": 1, "mix_norm": 2, "pre1": 3, "pre2": 4}
 
     def __init__(self, cfg: StackConfig, weights: dict, dtype: torch.dtype = torch.bfloat16, max_tokens: int = 512):
         self.cfg, self.dtype, self.weights, self.tp = cfg, dtype, weights, None
@@ -278,12 +331,19 @@ class StackModel(DecoderModel):
         c = _CConfig(n_layers=len(cfg.layers), d_model=cfg.d_model, vocab=cfg.vocab_size, max_seq=cfg.max_seq_len,
                      rms_eps=cfg.rms_norm_eps, tied=1 if cfg.tie_embeddings else 0)
         self._create(lib.ab2_model_create_stack, C.byref(c), specs, dtype_code(dtype), max_tokens)
+        check(lib.ab2_model_set_form(self._h, C.byref(cfg.c_form())))
         for name, w in weights.items():
             layer, leaf = -1, name
             if name.startswith("layers."):
                 layer, leaf = int(name.split(".")[1]), name.split(".")[2]
             if layer < 0 and leaf in ("embedding", "lm_head"):
                 check(lib.ab2_model_set_linear(self._h, -1, int(leaf == "lm_head"), w._h))
+            elif leaf == "loop_steps":
+                w = w.detach().to(torch.float32).contiguous()
+                check(lib.ab2_model_set_loop_steps(self._h, w.data_ptr()))
+            elif leaf == "table":
+                w = w.detach().to(torch.int32).contiguous()
+                check(lib.ab2_model_set_expert_table(self._h, layer, w.data_ptr()))
             elif layer < 0:
                 self._norm(-1, int(leaf == "embed_norm"), w)
             elif leaf in self.NORMS:

@@ -185,27 +185,44 @@ int ab2_embedding_forward(const ab2_qweight *table, const uint32_t *ids_dev, int
  * counterpart in the reference, whose decoder repeats one block. */
 typedef enum {
     AB2_MIX_ATTENTION = 0, /* grouped-query softmax attention over a sliding window */
-    AB2_MIX_LIGHTNING = 1  /* linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q */
+    AB2_MIX_LIGHTNING = 1, /* linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q */
+    AB2_MIX_LATENT = 2     /* causal softmax attention whose keys and values are projections of one cached latent */
 } ab2_mixer;
 typedef enum {
     AB2_FFN_NONE = 0,
-    AB2_FFN_MOE = 1 /* mixture of experts: sigmoid scores, the score multiplies the expert's input, clamped gated unit */
+    AB2_FFN_MOE = 1, /* mixture of experts over gated units */
+    AB2_FFN_POLY = 2 /* W_down act(W_up x), act(z) = a N(z) + b N(z^2) + c N(z^3) + e, powers element by element, N(z) = z / rms(z) over the row */
 } ab2_ffn;
+typedef enum {
+    AB2_GLU_CLAMPED = 0, /* g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1) */
+    AB2_GLU_SILU = 1     /* gate sigmoid(gate) up */
+} ab2_glu;
+typedef enum {
+    AB2_ROUTE_SIGMOID = 0, /* router: the largest sigmoid scores; the score multiplies what the expert reads */
+    AB2_ROUTE_TABLE = 1    /* no router: a table of token ids names the experts, each output weighs 1 / top */
+} ab2_routing;
 typedef struct {
     int mixer;          /* ab2_mixer */
     int heads, dim, vdim;
     int kv_heads;       /* attention */
     int window;         /* attention: keys a query sees, itself included; 0 = all */
-    int rot_dims;       /* attention: leading dimensions that are rotated, pairs (2i, 2i + 1); 0 = none */
+    int rot_dims;       /* attention: leading dimensions that are rotated, pairs (2i, 2i + 1); 0 = none.
+                           latent: rotated dimensions of a query besides the `dim` unrotated ones, and of the shared key part */
     double rot_base;
     int qk_norm;        /* attention: q and k divided by their root mean square after the rotation */
-    float scale;        /* attention: score = scale q.k */
+    float scale;        /* attention, latent: score = scale q.k */
     int v_mix;          /* attention: values are mixed with those of the stack's first layer that has this set */
     float v_lambda;     /* their weight: v <- (1 - lambda) v + lambda v_first */
     const float *decay; /* lightning: [heads], host memory, copied by the calls that take a spec */
     int ffn;            /* ab2_ffn */
     int experts, top, ff;
     float limit;        /* clamp of the gated unit */
+    int kv_rank;        /* latent: size of the cached latent */
+    int head_gate;      /* latent: a head's output is multiplied by the sigmoid of a gate value of its own */
+    int glu;            /* ab2_glu */
+    int routing;        /* ab2_routing */
+    int shared_ff;      /* mixture: width of an expert that runs for every token, 0 = none */
+    float poly[4];      /* AB2_FFN_POLY: a, b, c, e */
 } ab2_layer_spec;
 
 /* ---- KV cache --------------------------------------------------------------
@@ -285,6 +302,17 @@ int ab2_moe_workspace(const ab2_layer_spec *spec, int width, int tokens, ab2_dty
 int ab2_moe_forward(const ab2_layer_spec *spec, const ab2_qweight *router, const ab2_qweight *gate, const ab2_qweight *up,
                     const ab2_qweight *down, const void *x_dev, int tokens, ab2_dtype dtype, float *parts_dev, void *workspace_dev,
                     ab2_stream stream);
+/* Latent attention: proj_dev [nrows * S][stride] holds q (heads x (dim unrotated, rot_dims rotated)), the latent
+ * (kv_rank, normed here with norm_dev), the shared key part (rot_dims) and, with head_gate, heads gate values; ukv is
+ * the [heads (dim + vdim), kv_rank] up projection, head by head its key rows and its value rows; tables
+ * [positions][rot_dims / 2]; out_dev [nrows * S][heads vdim].  proj_dev may be rewritten.  workspace_dev holds
+ * ab2_latent_workspace bytes for nrows * S tokens and `positions` cached ones. */
+int ab2_latent_workspace(const ab2_layer_spec *spec, int tokens, int positions, ab2_dtype dtype, size_t *bytes);
+int ab2_latent_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *proj_dev, long long stride, const float *norm_dev,
+                         const ab2_qweight *ukv, const float *cos_dev, const float *sin_dev, float eps, void *out_dev,
+                         void *workspace_dev, size_t workspace_bytes, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
+/* out_dev [rows][n] = a N(z) + b N(z^2) + c N(z^3) + e with coef_host = {a, b, c, e} (AB2_FFN_POLY). */
+int ab2_poly_norm(const void *z_dev, void *out_dev, int rows, int n, const float *coef_host, float eps, ab2_dtype dtype, ab2_stream stream);
 
 /* ---- attention --------------------------------------------------------------
  * GroupedQueryAttention::forward_decode_batch attention step
@@ -351,18 +379,38 @@ int ab2_model_rope_tables(const ab2_model *m, const float **cos_dev, const float
 /* A decoder made of `n_layers` layer specs over one residual stream, which is kept in f32 whatever
  * `dtype` is (AB2_F32 or AB2_BF16): x = RMSNorm(embedding[token]); per layer x += RMSNorm(mixer(x)),
  * then x += RMSNorm(ffn(x)) where the layer has a feed-forward; logits = head . RMSNorm(x).  Of cfg
- * d_model, vocab, max_seq, rms_eps and tied are read.  Logits are f32.
+ * d_model, vocab, max_seq, rms_eps and tied are read.  Logits are f32.  ab2_model_set_form changes that frame.
  * Weights (FMT bf16, ab2_qweight_from_bf16) by ab2_model_set_linear, layer >= 0:
- *   which = 0  the mixer's input projections as one weight: attention q | k | v rows, lightning q | k | v | g rows
+ *   which = 0  the mixer's input projections as one weight: attention q | k | v rows, lightning q | k | v | g rows,
+ *              latent q | latent | shared key part | gate rows, then zero rows up to a multiple of 8
+ *   which = 1  latent: the up projection of keys and values (see ab2_latent_attention)
  *   which = 3  the mixer's output projection
  *   which = 4, 5, 6  the experts' gate, up ([experts * ff, d_model]) and down ([experts * d_model, ff]), expert by expert
+ *              (AB2_FFN_POLY: up [ff, d_model] and down [d_model, ff])
  *   which = 7  the router [experts, d_model]
+ *   which = 8, 9, 10  the shared expert's gate, up and down
  * Norms by ab2_model_set_norm, layer >= 0: which = 0 after the mixer, 1 after the feed-forward, 2 the lightning
- * mixer's own over heads * vdim; layer < 0: which = 0 the final norm, 1 the embedding's.
+ * mixer's own over heads * vdim or the latent's over kv_rank, 3 before the mixer, 4 before the feed-forward;
+ * layer < 0: which = 0 the final norm, 1 the embedding's.
  * The handle then serves ab2_model_finalize, ab2_model_forward*, ab2_model_decode_step* with caches of
  * ab2_kv_create_stack; offsets must be the cache lengths. */
 int ab2_model_create_stack(ab2_model **out, const ab2_model_config *cfg, const ab2_layer_spec *specs, ab2_dtype dtype,
                            int max_tokens);
+/* The frame around a stack's layers; call it before ab2_model_finalize.  Without it: embed_norm 1, the rest 0.
+ * A loop runs the layers loop_start .. loop_stop - 1 loop_times times in a row with the same weights; every run of a
+ * layer has a cache layer of its own, so the cache is created from the specs in the order of the runs.  Before pass t > 0
+ * the embedding (x as it was before the first layer) is added to x, and before every pass the t-th of the step vectors
+ * (ab2_model_set_loop_steps, [loop_times, d_model] f32). */
+typedef struct {
+    int embed_norm;     /* the embedding is normed */
+    int pre_norms;      /* sublayers read RMSNorm(x) instead of x */
+    int loop_start, loop_stop, loop_times;  /* loop_times 0: no loop */
+    float logit_softcap; /* logits z become softcap tanh(z / softcap); 0: they do not */
+} ab2_stack_form;
+int ab2_model_set_form(ab2_model *m, const ab2_stack_form *form);
+int ab2_model_set_loop_steps(ab2_model *m, const float *steps);
+/* AB2_ROUTE_TABLE: the experts of every token id, [vocab, top] i32 (host or device), copied. */
+int ab2_model_set_expert_table(ab2_model *m, int layer, const int *table);
 
 /* ---- tensor parallelism ------------------------------------------------------
  * Megatron-style sharding of the decoder over the GPUs of one box, one process

@@ -61,7 +61,7 @@ def test_configuration_reads_every_constant():
     assert a.scale == np.float32(0.3) and a.v_mix == 1 and a.v_lambda == float(w["l1.mix.vmix"])
     assert (specs[2].v_mix, specs[2].v_lambda, specs[2].ffn) == (0, 0.0, 0)
     assert (specs[1].experts, specs[1].top, specs[1].ff, specs[1].limit) == (4, 1, 40, np.float32(0.7))
-    assert C.sizeof(p._lib.LayerSpec) == 88
+    assert C.sizeof(p._lib.LayerSpec) == 120
     with pytest.raises(p.checkpoint.CheckpointError):
         p.tovelix.stack_config(dict(fx.VARIED, layers=[{"type": "other", "mixer": {}}]), w, 1)
     with pytest.raises(p.Ab2Error):
