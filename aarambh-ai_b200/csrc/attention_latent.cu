@@ -2,7 +2,8 @@
 // part that all heads share; head h's key is (W_uk,h c, key part) and its value W_uv,h c.
 //
 //   latent_prep_kernel     norm of the latent, rotation of queries and key part, store into the cache
-//   latent_attn_kernel     attention in the latent space on CUDA cores: f32 models, unusual sizes
+//   latent_tc_kernel       attention in the latent space on the tensor cores (attention_latent_tc.cu)
+//   latent_attn_kernel     the same on CUDA cores: f32 models, latents that shared memory cannot hold
 //   latent_merge_kernel    merge of the splits of a query's keys
 //
 // Decoding and short portions of a prompt never form keys and values: W_uk,h^T q_h is a query against
@@ -230,8 +231,15 @@ bool expandable(int dim, int rot, int rank, int vdim, ab2_dtype dtype) {
 
 // Attention of a.S queries per row in the latent space: qx [T][H][kds] -> ox [T][H][rank].
 template <typename T>
-int latent_space_attention(LatentArgs a, const T *qx, T *ox, int nrows, int max_len, cudaStream_t s) {
+int latent_space_attention(const ab2_kv *kv, LatentArgs a, const T *qx, T *ox, int nrows, int max_len, cudaStream_t s) {
     const KvLayer &l = a.kv.l;
+    if (sizeof(T) == 2 && latent_tc_serves(a.rank, l.kds)) {
+        int rc = latent_tc_attention(a, (const __nv_bfloat16 *)qx, (__nv_bfloat16 *)ox, kv->B, nrows, max_len, s);
+        if (rc != AB2_OK || a.nsplit == 1) return rc;
+        cudaError_t e = launch_kernel(latent_merge_kernel<T>, dim3(nrows * a.S * a.H), dim3(128), 0, s, a, ox);
+        if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "latent attention launch failed: %s", cudaGetErrorString(e));
+        return AB2_OK;
+    }
     const int tokens = nrows * a.S, groups = (a.H + LA_REP - 1) / LA_REP, units = groups * tokens;
     a.nsplit = 1;
     if (units < device_sm_count()) {  // the splits' sums fit the scratch: LATENT_PART_TILES * LATENT_ROWS rows
@@ -271,7 +279,7 @@ int launch_latent(const ab2_kv *kv, LatentArgs a, int nrows, int max_len, ab2_dt
         lin.x = a.proj; lin.ldx = a.stride; lin.xb = D;
         lin.y = qx; lin.ldy = (long long)a.H * l.kds; lin.yb = l.kds; lin.epi = LIN_STORE;
         int rc = linear_dense(lin, dtype, s);
-        if (rc == AB2_OK) rc = latent_space_attention<T>(a, qx, ox, nrows, max_len, s);
+        if (rc == AB2_OK) rc = latent_space_attention<T>(kv, a, qx, ox, nrows, max_len, s);
         if (rc != AB2_OK) return rc;
         lin.w = a.ukv + (size_t)a.dim * a.rank; lin.wb = (long long)(a.dim + a.vdim) * a.rank; lin.N = a.vdim; lin.K = a.rank;
         lin.x = ox; lin.ldx = (long long)a.H * a.rank; lin.xb = a.rank;

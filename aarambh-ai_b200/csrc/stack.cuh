@@ -76,6 +76,10 @@ size_t latent_workspace(int H, int dim, int rot, int rank, int vdim, int tokens,
 int latent_attention(const ab2_kv *kv, LatentArgs a, int nrows, int max_len, ab2_dtype dtype, cudaStream_t s);
 // absorb[h][r][d] = ukv[h][d][r] over the key rows
 int latent_absorb_weights(const __nv_bfloat16 *ukv, __nv_bfloat16 *absorb, int H, int dim, int vdim, int rank, cudaStream_t s);
+// The bf16 kernel of attention in the latent space (attention_latent_tc.cu): qx [nrows * S][H][kds] to
+// ox [nrows * S][H][rank], or with a.nsplit > 1, which it chooses, to the splits' sums in a.part_acc, a.part_ml.
+bool latent_tc_serves(int rank, int kds);
+int latent_tc_attention(LatentArgs &a, const __nv_bfloat16 *qx, __nv_bfloat16 *ox, int cache_rows, int nrows, int max_len, cudaStream_t s);
 constexpr int LATENT_ROWS = 32;    // (token, head) rows of a CTA of the decode kernel
 constexpr int LATENT_PART_TILES = 320;  // row tiles x splits that the cache's scratch holds
 static inline size_t latent_part_bytes(const ab2_layer_spec &sp) { return (size_t)LATENT_PART_TILES * LATENT_ROWS * sp.kv_rank * 4; }
