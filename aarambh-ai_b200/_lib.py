@@ -90,7 +90,7 @@ SIGNATURES = {
     "ab2_moe_workspace": ([_p, _i, _i, _i, C.POINTER(C.c_size_t)], _i),
     "ab2_moe_forward": ([_p, _p, _p, _p, _p, _p, _i, _i, _p, _p, _p], _i),
     "ab2_latent_workspace": ([_p, _i, _i, _i, C.POINTER(C.c_size_t)], _i),
-    "ab2_latent_attention": ([_p, _i, _p, _p, C.c_longlong, _p, _p, _p, _p, _f, _p, _p, C.c_size_t, _i, _i, _i, _i, _p], _i),
+    "ab2_latent_attention": ([_p, _i, _p, _p, C.c_longlong, _p, _p, _p, _p, _f, _p, _p, C.c_size_t, _i, _i, _i, _i, _i, _p], _i),
     "ab2_poly_norm": ([_p, _p, _i, _i, C.POINTER(_f), _f, _i, _p], _i),
     "ab2_attention_decode": ([_p, _i, _p, _p, _i, _i, _f, _i, _p], _i),
     "ab2_attention_decode_static": ([_p, _i, _p, _p, _i, _i, _f, _i, _p], _i),

@@ -2,6 +2,7 @@
 // part that all heads share; head h's key is (W_uk,h c, key part) and its value W_uv,h c.
 //
 //   latent_prep_kernel     norm of the latent, rotation of queries and key part, store into the cache
+//   latent_absorb_kernel   the same and the queries against the latents, in one launch (bf16)
 //   latent_tc_kernel       attention in the latent space on the tensor cores (attention_latent_tc.cu)
 //   latent_attn_kernel     the same on CUDA cores: f32 models, latents that shared memory cannot hold
 //   latent_merge_kernel    merge of the splits of a query's keys
@@ -164,20 +165,39 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(LatentArgs a, const T 
     }
 }
 
-// One CTA per (token, head): ox = sum of the splits' latents, weighted by 2^(m - max), over the sum of
-// their weights.
-template <typename T>
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, T *ox) {
+// grid (token-head rows, ceil(rank / (1024 / G))): ox = sum of the splits' latents, weighted by 2^(m - max), over
+// the sum of their weights.  A thread takes four dimensions of every G-th split, eight splits at most.
+template <typename T, int G>
+__global__ void __launch_bounds__(256) latent_merge_kernel(LatentArgs a, T *ox) {
+    constexpr int LANES = 256 / G;
     __shared__ float wt[AB2_KV_MAX_SPLITS];
+    __shared__ float4 red[G][LANES];
     pdl_wait();
     pdl_launch_dependents();
+    const int group = threadIdx.x / LANES, lane = threadIdx.x % LANES;
     const size_t r = blockIdx.x, p0 = r * a.nsplit;
+    const int d0 = (blockIdx.y * LANES + lane) * 4, nd = min(4, a.rank - d0);
+    const float *src = a.part_acc + p0 * a.rank + d0;
+    float4 v[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+        const int sp = group + G * k;
+        v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (sp < a.nsplit && nd == 4 && (a.rank & 3) == 0) v[k] = *reinterpret_cast<const float4 *>(src + (size_t)sp * a.rank);
+    }
+    if ((a.rank & 3) != 0)
+        for (int k = 0; k < 8 && group + G * k < a.nsplit; ++k) {
+            const float *q = src + (size_t)(group + G * k) * a.rank;
+            if (nd > 0) v[k].x = q[0];
+            if (nd > 1) v[k].y = q[1];
+            if (nd > 2) v[k].z = q[2];
+            if (nd > 3) v[k].w = q[3];
+        }
     if (threadIdx.x < 32) {
-        const int lane = threadIdx.x;
         float m[2], ls[2], top = -INFINITY, sum = 0.f;
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
-            const int sp = lane + 32 * k;
+            const int sp = threadIdx.x + 32 * k;
             m[k] = sp < a.nsplit ? a.part_ml[(p0 + sp) * 2] : -INFINITY;
             ls[k] = sp < a.nsplit ? a.part_ml[(p0 + sp) * 2 + 1] : 0.f;
             top = fmaxf(top, m[k]);
@@ -192,19 +212,165 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, T *ox) 
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
 #pragma unroll
-        for (int k = 0; k < 2; ++k)
-            if (lane + 32 * k < a.nsplit) wt[lane + 32 * k] = m[k] / sum;
+        for (int k = 0; k < 2; ++k) wt[threadIdx.x + 32 * k] = m[k] / sum;
     }
     __syncthreads();
-    for (int d = threadIdx.x; d < a.rank; d += 128) {
-        float v = 0.f;
-#pragma unroll 8
-        for (int k = 0; k < a.nsplit; ++k) {
-            const float w = wt[k];
-            if (w != 0.f) v = fmaf(w, a.part_acc[(p0 + k) * a.rank + d], v);  // an empty split has written nothing
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+        const float w = group + G * k < a.nsplit ? wt[group + G * k] : 0.f;
+        if (w != 0.f) {  // an empty split has written nothing
+            s.x = fmaf(w, v[k].x, s.x); s.y = fmaf(w, v[k].y, s.y); s.z = fmaf(w, v[k].z, s.z); s.w = fmaf(w, v[k].w, s.w);
         }
-        ox[r * a.rank + d] = from_f32<T>(v);
     }
+    if (G > 1) {
+        red[group][lane] = s;
+        __syncthreads();
+        if (group > 0) return;
+#pragma unroll
+        for (int g = 1; g < G; ++g) {
+            const float4 q = red[g][lane];
+            s.x += q.x; s.y += q.y; s.z += q.z; s.w += q.w;
+        }
+    }
+    T *dst = ox + r * a.rank + d0;
+    if (nd > 0) dst[0] = from_f32<T>(s.x);
+    if (nd > 1) dst[1] = from_f32<T>(s.y);
+    if (nd > 2) dst[2] = from_f32<T>(s.z);
+    if (nd > 3) dst[3] = from_f32<T>(s.w);
+}
+
+template <typename T>
+cudaError_t launch_merge(const LatentArgs &a, T *ox, int rows, cudaStream_t s) {
+    if (a.nsplit <= 8 && a.rank > 256) return launch_kernel(latent_merge_kernel<T, 1>, dim3(rows, (a.rank + 1023) / 1024), dim3(256), 0, s, a, ox);
+    if (a.nsplit <= 16) return launch_kernel(latent_merge_kernel<T, 2>, dim3(rows, (a.rank + 511) / 512), dim3(256), 0, s, a, ox);
+    return launch_kernel(latent_merge_kernel<T, 8>, dim3(rows, (a.rank + 127) / 128), dim3(256), 0, s, a, ox);
+}
+
+// bf16, few tokens: absorbed queries, rotations, norm and store in one launch.  grid (ceil(rank / 128), token
+// tiles of 8 NT, H + 1), 256 threads.  A layer z < H of the grid multiplies W_uk,h^T by the head's unrotated
+// queries: a warp owns 16 latent dimensions over the whole (short) sum, its fragments read as in
+// gemv_bf16.cu; its first CTA rotates the head's queries.  Layer H norms the latents, rotates the key
+// parts and stores both.  KC chunks of 32 unrotated dimensions.
+__device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int KC, int NT>
+__global__ void __launch_bounds__(256) latent_absorb_kernel(LatentArgs a, __nv_bfloat16 *qx, int tokens) {
+    __shared__ __align__(16) __nv_bfloat16 tile[8 * NT][128 + 8];
+    const KvLayer &l = a.kv.l;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
+    const int h = blockIdx.z, m0 = blockIdx.y * 8 * NT, r0 = blockIdx.x * 128, D = a.dim + a.rot, half = a.rot >> 1;
+    const __nv_bfloat16 *proj = (const __nv_bfloat16 *)a.proj;
+    auto position = [&](int t, int &row) {
+        row = kv_row(a.kv, a.row0, t / a.S);
+        return a.kv.lens[row] + t % a.S;
+    };
+    if (h == a.H) {
+        pdl_wait();
+        pdl_launch_dependents();
+        for (int t = m0 + blockIdx.x * 8 + warp; t < min(tokens, m0 + 8 * NT); t += 8 * gridDim.x) {
+            int row;
+            const int pos = position(t, row);
+            const __nv_bfloat16 *src = proj + t * a.stride + (size_t)a.H * D;
+            __nv_bfloat16 *dst = (__nv_bfloat16 *)l.k + ((size_t)row * l.cap + pos) * l.kds;  // capacity is checked on the host
+            uint4 v[4];  // a lane's values, eight at a time; rank is a multiple of 8 and 1024 at most
+#pragma unroll
+            for (int k = 0; k < 4; ++k) v[k] = (lane + 32 * k) * 8 < a.rank ? reinterpret_cast<const uint4 *>(src)[lane + 32 * k] : make_uint4(0u, 0u, 0u, 0u);
+            float sum = 0.f;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const uint32_t w[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float lo = __uint_as_float(w[e] << 16), hi = __uint_as_float(w[e] & 0xffff0000u);
+                    sum = fmaf(lo, lo, fmaf(hi, hi, sum));
+                }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            const float inv = 1.f / sqrtf(sum / (float)a.rank + a.eps);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const int d = (lane + 32 * k) * 8;
+                if (d >= a.rank) continue;
+                const float4 na = reinterpret_cast<const float4 *>(a.norm_w + d)[0], nb = reinterpret_cast<const float4 *>(a.norm_w + d)[1];
+                const uint32_t w[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+                const float nw[8] = {na.x, na.y, na.z, na.w, nb.x, nb.y, nb.z, nb.w};
+                uint32_t o[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const __nv_bfloat162 q = __floats2bfloat162_rn(__uint_as_float(w[e] << 16) * inv * nw[2 * e], __uint_as_float(w[e] & 0xffff0000u) * inv * nw[2 * e + 1]);
+                    o[e] = *reinterpret_cast<const uint32_t *>(&q);
+                }
+                *reinterpret_cast<uint4 *>(dst + d) = make_uint4(o[0], o[1], o[2], o[3]);
+            }
+            for (int j = lane; j < half; j += 32) {
+                const float u = __bfloat162float(src[a.rank + 2 * j]), v = __bfloat162float(src[a.rank + 2 * j + 1]);
+                const float cs = a.cos_t[(size_t)pos * half + j], sn = a.sin_t[(size_t)pos * half + j];
+                dst[a.rank + 2 * j] = __float2bfloat16_rn(u * cs - v * sn);
+                dst[a.rank + 2 * j + 1] = __float2bfloat16_rn(v * cs + u * sn);
+            }
+        }
+        return;
+    }
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    const int ra = r0 + warp * 16 + g;
+    const __nv_bfloat16 *w = a.absorb + (size_t)h * a.rank * a.dim + c * 8;
+    uint4 va[KC], vb[KC];
+#pragma unroll
+    for (int k = 0; k < KC; ++k) {
+        const bool in = k * 32 + c * 8 < a.dim;  // dim is a multiple of 8
+        va[k] = in ? *reinterpret_cast<const uint4 *>(w + (size_t)min(ra, a.rank - 1) * a.dim + k * 32) : zero;
+        vb[k] = in ? *reinterpret_cast<const uint4 *>(w + (size_t)min(ra + 8, a.rank - 1) * a.dim + k * 32) : zero;
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    float acc[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+        acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+        const int t = m0 + j * 8 + g;
+        const __nv_bfloat16 *x = proj + (size_t)min(t, tokens - 1) * a.stride + (size_t)h * D + c * 8;
+#pragma unroll
+        for (int k = 0; k < KC; ++k) {
+            const uint4 b = k * 32 + c * 8 < a.dim ? *reinterpret_cast<const uint4 *>(x + k * 32) : zero;
+            mma_bf16(acc[j], va[k].x, vb[k].x, va[k].y, vb[k].y, b.x, b.y);
+            mma_bf16(acc[j], va[k].z, vb[k].z, va[k].w, vb[k].w, b.z, b.w);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) tile[j * 8 + 2 * c + (i & 1)][warp * 16 + g + 8 * (i >> 1)] = __float2bfloat16_rn(acc[j][i]);
+    }
+    // this head's queries, rotated behind the latent part, and the padding of a row: the CTAs of a head share its tokens
+    const int pairs = half + ((l.kds - a.rank - a.rot) >> 1);  // rotated ones, then padding (rank, rot and kds are even)
+    for (int i = blockIdx.x * 256 + threadIdx.x; i < 8 * NT * pairs; i += 256 * gridDim.x) {
+        const int t = m0 + i / pairs, j = i % pairs;
+        if (t >= tokens) break;
+        float u = 0.f, v = 0.f, cs = 0.f, sn = 0.f;
+        if (j < half) {
+            int row;
+            const int pos = position(t, row);
+            const __nv_bfloat162 q = *reinterpret_cast<const __nv_bfloat162 *>(proj + t * a.stride + (size_t)h * D + a.dim + 2 * j);
+            u = __low2float(q); v = __high2float(q); cs = a.cos_t[(size_t)pos * half + j]; sn = a.sin_t[(size_t)pos * half + j];
+        }
+        *reinterpret_cast<__nv_bfloat162 *>(qx + ((size_t)t * a.H + h) * l.kds + a.rank + 2 * j) = __floats2bfloat162_rn(u * cs - v * sn, v * cs + u * sn);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 8 * NT * 16; i += 256) {  // 8 dimensions each
+        const int t = m0 + i / 16, d = r0 + (i % 16) * 8;
+        if (t < tokens && d < a.rank) *reinterpret_cast<uint4 *>(qx + ((size_t)t * a.H + h) * l.kds + d) = *reinterpret_cast<const uint4 *>(&tile[i / 16][(i % 16) * 8]);
+    }
+}
+
+template <int KC>
+cudaError_t launch_absorb(const LatentArgs &a, __nv_bfloat16 *qx, int tokens, cudaStream_t s) {
+    const int nt = tokens <= 8 ? 1 : tokens <= 16 ? 2 : 4;
+    const dim3 grid((a.rank + 127) / 128, (tokens + 8 * nt - 1) / (8 * nt), a.H + 1);
+    if (nt == 1) return launch_kernel(latent_absorb_kernel<KC, 1>, grid, dim3(256), 0, s, a, qx, tokens);
+    if (nt == 2) return launch_kernel(latent_absorb_kernel<KC, 2>, grid, dim3(256), 0, s, a, qx, tokens);
+    return launch_kernel(latent_absorb_kernel<KC, 4>, grid, dim3(256), 0, s, a, qx, tokens);
 }
 
 __global__ void absorb_weights_kernel(const __nv_bfloat16 *ukv, __nv_bfloat16 *absorb, int dim, int vdim, int rank) {
@@ -236,7 +402,7 @@ int latent_space_attention(const ab2_kv *kv, LatentArgs a, const T *qx, T *ox, i
     if (sizeof(T) == 2 && latent_tc_serves(a.rank, l.kds)) {
         int rc = latent_tc_attention(a, (const __nv_bfloat16 *)qx, (__nv_bfloat16 *)ox, kv->B, nrows, max_len, s);
         if (rc != AB2_OK || a.nsplit == 1) return rc;
-        cudaError_t e = launch_kernel(latent_merge_kernel<T>, dim3(nrows * a.S * a.H), dim3(128), 0, s, a, ox);
+        cudaError_t e = launch_merge<T>(a, ox, nrows * a.S * a.H, s);
         if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "latent attention launch failed: %s", cudaGetErrorString(e));
         return AB2_OK;
     }
@@ -257,7 +423,7 @@ int latent_space_attention(const ab2_kv *kv, LatentArgs a, const T *qx, T *ox, i
         configured[dev] = true;
     }
     cudaError_t e = launch_kernel(latent_attn_kernel<T>, dim3(a.nsplit, groups, tokens), dim3(256), smem, s, a, qx, ox);
-    if (e == cudaSuccess && a.nsplit > 1) e = launch_kernel(latent_merge_kernel<T>, dim3(tokens * a.H), dim3(128), 0, s, a, ox);
+    if (e == cudaSuccess && a.nsplit > 1) e = launch_merge<T>(a, ox, tokens * a.H, s);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "latent attention launch failed: %s", cudaGetErrorString(e));
     return AB2_OK;
 }
@@ -270,7 +436,13 @@ int launch_latent(const ab2_kv *kv, LatentArgs a, int nrows, int max_len, ab2_dt
     const size_t head_bytes = (size_t)max_len * (a.dim + a.vdim) * 2;  // keys and values of one head
     const bool expand = a.S >= EXPAND_TOKENS && expandable(a.dim, a.rot, a.rank, a.vdim, dtype) && D % 2 == 0 && a.stride % 8 == 0 && a.work_bytes >= head_bytes;
     T *qx = (T *)a.work, *ox = (T *)((char *)a.work + up256((size_t)T_ * a.H * l.kds * sizeof(T)));
-    cudaError_t e = launch_kernel(latent_prep_kernel<T>, dim3(a.S, nrows), dim3(256), 0, s, a, expand ? (T *)nullptr : qx);
+    const bool fused = !expand && dtype == AB2_BF16 && a.rank % 8 == 0 && a.dim % 8 == 0 && a.dim <= 256 && a.rot % 8 == 0 && a.stride % 8 == 0;
+    cudaError_t e;
+    if (!fused) e = launch_kernel(latent_prep_kernel<T>, dim3(a.S, nrows), dim3(256), 0, s, a, expand ? (T *)nullptr : qx);
+    else if (a.dim <= 32) e = launch_absorb<1>(a, (__nv_bfloat16 *)qx, T_, s);
+    else if (a.dim <= 64) e = launch_absorb<2>(a, (__nv_bfloat16 *)qx, T_, s);
+    else if (a.dim <= 128) e = launch_absorb<4>(a, (__nv_bfloat16 *)qx, T_, s);
+    else e = launch_absorb<8>(a, (__nv_bfloat16 *)qx, T_, s);
     if (e != cudaSuccess) return fail(AB2_ERR_CUDA, "latent preparation launch failed: %s", cudaGetErrorString(e));
     LinArgs lin = {};
     lin.M = T_; lin.batch = a.H;
@@ -278,7 +450,7 @@ int launch_latent(const ab2_kv *kv, LatentArgs a, int nrows, int max_len, ab2_dt
         lin.w = a.absorb; lin.wb = (long long)a.rank * a.dim; lin.N = a.rank; lin.K = a.dim;
         lin.x = a.proj; lin.ldx = a.stride; lin.xb = D;
         lin.y = qx; lin.ldy = (long long)a.H * l.kds; lin.yb = l.kds; lin.epi = LIN_STORE;
-        int rc = linear_dense(lin, dtype, s);
+        int rc = fused ? (int)AB2_OK : linear_dense(lin, dtype, s);
         if (rc == AB2_OK) rc = latent_space_attention<T>(kv, a, qx, ox, nrows, max_len, s);
         if (rc != AB2_OK) return rc;
         lin.w = a.ukv + (size_t)a.dim * a.rank; lin.wb = (long long)(a.dim + a.vdim) * a.rank; lin.N = a.vdim; lin.K = a.rank;

@@ -615,7 +615,7 @@ AB2_API int ab2_latent_workspace(const ab2_layer_spec *spec, int tokens, int pos
 
 AB2_API int ab2_latent_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *proj_dev, long long stride, const float *norm_dev,
                                  const ab2_qweight *ukv, const float *cos_dev, const float *sin_dev, float eps, void *out_dev,
-                                 void *workspace_dev, size_t workspace_bytes, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream) {
+                                 void *workspace_dev, size_t workspace_bytes, int reuse, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream) {
     STEP(check_mixer_call(kv, layer, spec, AB2_MIX_LATENT, proj_dev, out_dev, S, row0, nrows, dtype));
     const int H = spec->heads, D = spec->dim + spec->rot_dims;
     AB2_REQUIRE(norm_dev && ukv && workspace_dev && (spec->rot_dims == 0 || (cos_dev && sin_dev)), AB2_ERR_BAD_ARG, "null argument");
@@ -625,7 +625,7 @@ AB2_API int ab2_latent_attention(ab2_kv *kv, int layer, const ab2_layer_spec *sp
     AB2_REQUIRE(workspace_bytes >= absorb + latent_workspace(H, spec->dim, spec->rot_dims, spec->kv_rank, spec->vdim, nrows * S, 1, dtype), AB2_ERR_BAD_SHAPE,
                 "workspace of %zu bytes is too small", workspace_bytes);
     __nv_bfloat16 *absorbed = (__nv_bfloat16 *)workspace_dev;
-    STEP(latent_absorb_weights((const __nv_bfloat16 *)ukv->codes, absorbed, H, spec->dim, spec->vdim, spec->kv_rank, (cudaStream_t)stream));
+    if (!reuse) STEP(latent_absorb_weights((const __nv_bfloat16 *)ukv->codes, absorbed, H, spec->dim, spec->vdim, spec->kv_rank, (cudaStream_t)stream));
     LatentArgs a = {};
     a.kv = kv_layer_view(kv, layer);
     a.proj = proj_dev; a.stride = stride; a.S = S; a.row0 = row0; a.H = H; a.dim = spec->dim; a.rot = spec->rot_dims; a.rank = spec->kv_rank;

@@ -58,7 +58,6 @@ __device__ __forceinline__ bool bar_wait(uint64_t *b, uint32_t parity, volatile 
     *failed = 1;
     return false;
 }
-
 __device__ __forceinline__ void bulk_copy(void *dst, const void *src, uint32_t bytes, uint64_t *bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n" ::
                      "r"(sptr(dst)), "l"(src), "r"(bytes), "r"(sptr(bar)) : "memory");

@@ -177,9 +177,10 @@ def lightning_attention(cache, cfg, layer: int, qkv: torch.Tensor, powers: torch
 
 
 def latent_attention(cache, cfg, layer: int, proj: torch.Tensor, norm: torch.Tensor, ukv, tables, eps: float, row0: int = 0,
-                     workspace: torch.Tensor | None = None) -> torch.Tensor:
+                     workspace: torch.Tensor | None = None, reuse: bool = False) -> torch.Tensor:
     """proj [rows, S, stride] (overwritten): heads (dim + rot_dims) queries | latent | shared key part | gates;
-    ``ukv`` the keys' and values' up projection (``QuantLinear``) -> [rows, S, heads vdim]."""
+    ``ukv`` the keys' and values' up projection (``QuantLinear``) -> [rows, S, heads vdim].  With ``reuse`` the
+    workspace is that of an earlier call with the same ``ukv``."""
     proj = _cuda(proj, "proj")
     specs, _keep = cfg.c_specs(cfg.runs())
     sp = specs[layer]
@@ -192,7 +193,7 @@ def latent_attention(cache, cfg, layer: int, proj: torch.Tensor, norm: torch.Ten
     cos, sin = tables if tables is not None else (None, None)
     check(lib.ab2_latent_attention(cache._h, layer, C.byref(sp), proj.data_ptr(), stride, norm.data_ptr(), ukv._h,
                                    cos.data_ptr() if cos is not None else None, sin.data_ptr() if sin is not None else None, float(eps),
-                                   out.data_ptr(), workspace.data_ptr(), workspace.numel(), S, row0, rows, dtype_code(proj.dtype), stream_ptr()))
+                                   out.data_ptr(), workspace.data_ptr(), workspace.numel(), int(reuse), S, row0, rows, dtype_code(proj.dtype), stream_ptr()))
     return out
 
 

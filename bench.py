@@ -449,61 +449,141 @@ def time_model(pkg, torch, model, vocab, kv_dtype, batches, prompts, steps, ctx=
     return out
 
 
-def tovelix_record(args):
-    """`--model tovelix`: decode and prefill throughput of the Tovelix stack beside the dense decoder of
-    equal width, depth, heads and active feed-forward width."""
+# Vipelix at the same sizes: six layers of which two are looped over twice (eight runs), the first with a
+# dense feed-forward of the experts' active width.  "tovelix" is the closest existing model at equal size: eight
+# layers of softmax attention over the whole context, as many active expert weights, the same number format.
+VIPELIX = {
+    "w2048": dict(width=2048, layers=6, loop=(2, 4, 2), heads=16, dim=128, rot=64, vdim=128, rank=512, experts=32, top=3, ff=1024, shared=1024, dense=6144),
+    "w4096": dict(width=4096, layers=6, loop=(2, 4, 2), heads=32, dim=128, rot=64, vdim=128, rank=512, experts=8, top=1, ff=7168, shared=7168, dense=21504),
+}
+
+
+def build_vipelix(pkg, torch, c, max_tokens, max_seq, vocab=32000):
+    gen = torch.Generator(device="cuda").manual_seed(0)
+
+    def lin(n, k):
+        w = torch.empty((n, k), dtype=torch.bfloat16, device="cuda").normal_(generator=gen)
+        return pkg.QuantLinear.from_bf16(w.mul_(k ** -0.5))
+
+    d, H, E, top, ff, sh = c["width"], c["heads"], c["experts"], c["top"], c["ff"], c["shared"]
+    ones = torch.ones(max(d, c["rank"]), device="cuda")
+    mix = pkg.LatentMixer(H, c["dim"], c["rot"], c["vdim"], c["rank"], (c["dim"] + c["rot"]) ** -0.5, 10000.0, True)
+    weights = {"embedding": lin(vocab, d), "final_norm": ones[:d], "loop_steps": torch.randn(c["loop"][2], d)}
+    layers = []
+    for i in range(c["layers"]):
+        q = f"layers.{i}."
+        n = H * (c["dim"] + c["rot"]) + c["rank"] + c["rot"] + H
+        weights.update({q + "in": lin(-(-n // 8) * 8, d), q + "ukv": lin(H * (c["dim"] + c["vdim"]), c["rank"]), q + "out": lin(d, H * c["vdim"]),
+                        q + "mix_norm": ones[:c["rank"]]})
+        for norm in ("pre1", "norm1", "pre2", "norm2"):
+            weights[q + norm] = ones[:d]
+        if i == 0:
+            layers.append((mix, pkg.PolyFfn(c["dense"], (0.5, 0.3, 0.2, 0.0))))
+            weights[q + "up"], weights[q + "down"] = lin(c["dense"], d), lin(d, c["dense"])
+            continue
+        layers.append((mix, pkg.MoeFfn(E, top, ff, glu="silu", routing="table", shared_ff=sh)))
+        weights[q + "table"] = torch.rand((vocab, E), generator=torch.Generator().manual_seed(i)).topk(top, 1).indices.to(torch.int32)
+        weights[q + "gate"], weights[q + "up"], weights[q + "down"] = lin(E * ff, d), lin(E * ff, d), lin(E * d, ff)
+        weights[q + "shared_gate"], weights[q + "shared_up"], weights[q + "shared_down"] = lin(sh, d), lin(sh, d), lin(d, sh)
+    cfg = pkg.StackConfig(d, vocab, layers, max_seq, embed_norm=False, pre_norms=True, loop=c["loop"], logit_softcap=30.0)
+    return pkg.StackModel(cfg, weights, torch.bfloat16, max_tokens)
+
+
+def vipelix_runs(c):
+    """Runs of the dense layer and of the others in a pass."""
+    start, stop, times = c["loop"]
+    runs = [i for i in range(c["layers"]) for _ in range(times if start <= i < stop else 1)]
+    return runs.count(0), len(runs) - runs.count(0)
+
+
+def vipelix_step_bytes(c, batch, ctx, vocab=32000):
+    """Algorithmic bytes of a decode step: the weights of every run once (experts: as many as the batch can
+    reach) and the cached rows."""
+    d, H, r = c["width"], c["heads"], c["rank"]
+    hit = c["experts"] * (1 - (1 - c["top"] / c["experts"]) ** batch)
+    mix = 2 * ((H * (c["dim"] + c["rot"]) + r + c["rot"] + H) * d + H * (c["dim"] + c["vdim"]) * r + H * c["vdim"] * d) + batch * ctx * 2 * (r + c["rot"])
+    dense, moe = vipelix_runs(c)
+    return (dense + moe) * mix + dense * 4 * d * c["dense"] + moe * 6 * d * (hit * c["ff"] + c["shared"]) + 2 * vocab * d
+
+
+def vipelix_prefill_flops(c, S, vocab=32000):
+    d, H, r = c["width"], c["heads"], c["rank"]
+    mix = 2 * S * ((H * (c["dim"] + c["rot"]) + r + c["rot"] + H) * d + H * (c["dim"] + c["vdim"]) * r + H * c["vdim"] * d)
+    mix += H * (c["dim"] + c["rot"] + c["vdim"]) * S * (S + 1)
+    dense, moe = vipelix_runs(c)
+    return (dense + moe) * mix + dense * 4 * S * d * c["dense"] + moe * 6 * S * d * (c["top"] * c["ff"] + c["shared"]) + 2 * vocab * d
+
+
+def dense_like_tovelix(pkg, torch, c, prompts, vocab):
+    """The dense decoder of a Tovelix size: model, cache type, bytes of a step, FLOPs of a prompt."""
+    n = len(c["layers"])
+    dc = dict(n_layers=n, d_model=c["width"], n_heads=c["heads"], n_kv_heads=c["kv_heads"], head_dim=128,
+              ffn_hidden=c["top"] * c["ff"], vocab=vocab, max_seq=max(prompts) + 512)
+    mc, weights = build_large(pkg, torch, dc)
+    model = pkg.AarambhModel(mc, weights, dtype=torch.bfloat16, max_tokens=max(prompts))
+    return model, "int8", lambda B: step_weight_bytes(dc) + B * PROMPT * kv_bytes_per_token(dc), \
+        lambda S: 2.0 * S * sum(a * b for a, b in linear_shapes(dc).values()) * n + 2.0 * vocab * c["width"] + n * 2.0 * c["heads"] * 128 * S * (S + 1)
+
+
+def tovelix_like_vipelix(pkg, torch, c, prompts, vocab):
+    """The Tovelix stack of a Vipelix size: attention over the whole context in every layer."""
+    t = dict(width=c["width"], layers="A" * sum(vipelix_runs(c)), heads=c["heads"], kv_heads=c["heads"] // 4, window=max(prompts) + 512,
+             experts=c["experts"], top=c["top"] + c["shared"] // c["ff"], ff=c["ff"])
+    return build_tovelix(pkg, torch, t, max(prompts), max(prompts) + 512, vocab), "bf16", lambda B: tovelix_step_bytes(t, B, PROMPT), \
+        lambda S: tovelix_prefill_flops(t, S)
+
+
+STACKS = {"tovelix": (TOVELIX, build_tovelix, tovelix_step_bytes, tovelix_prefill_flops, "dense_w4a16", dense_like_tovelix),
+          "vipelix": (VIPELIX, build_vipelix, vipelix_step_bytes, vipelix_prefill_flops, "tovelix", tovelix_like_vipelix)}
+
+
+def stack_record(args):
+    """`--model tovelix` / `--model vipelix`: decode and prefill throughput of a layer stack beside the closest
+    existing model of equal size."""
     import torch
     torch.cuda.set_device(0)
     from __graft_entry__ import import_package
     pkg = import_package()
     peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
     hbm, tf = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    table, build, step_bytes, prefill_flops, like_name, like = STACKS[args.model]
     batches, prompts, vocab = (1, 8, 32), (512, 2048, 8192), 32000
     sizes = {}
     clocks = ClockSampler(0)
-    for name, c in TOVELIX.items():
+
+    def measure(model, kv, byt, flops):
+        with clocks:
+            t = time_model(pkg, torch, model, vocab, kv, batches, prompts, args.steps)
+        return {f"batch{B}": {"ms": round(ms, 4), "tok_s": round(B * 1e3 / ms, 1), "hbm_frac": round(byt(B) / ms / 1e6 / hbm, 4)}
+                for B, ms in t["decode"].items()}, \
+               {f"{S}": {"ms": round(ms, 3), "tok_s": round(S * 1e3 / ms, 1), "bf16_frac": round(flops(S) / ms / 1e9 / tf, 4)}
+                for S, ms in t["prefill"].items()}
+
+    for name, c in table.items():
         if args.size not in ("all", name):
             continue
-        model = build_tovelix(pkg, torch, c, max(prompts), max(prompts) + 512, vocab)
-        with clocks:
-            t = time_model(pkg, torch, model, vocab, "bf16", batches, prompts, args.steps)
+        model = build(pkg, torch, c, max(prompts), max(prompts) + 512, vocab)
+        decode, prefill = measure(model, "bf16", lambda B: step_bytes(c, B, PROMPT), lambda S: prefill_flops(c, S))
         del model
         torch.cuda.empty_cache()
-        n = len(c["layers"])
-        dc = dict(n_layers=n, d_model=c["width"], n_heads=c["heads"], n_kv_heads=c["kv_heads"], head_dim=128,
-                  ffn_hidden=c["top"] * c["ff"], vocab=vocab, max_seq=max(prompts) + 512)
-        mc, weights = build_large(pkg, torch, dc)
-        dense = pkg.AarambhModel(mc, weights, dtype=torch.bfloat16, max_tokens=max(prompts))
-        with clocks:
-            u = time_model(pkg, torch, dense, vocab, "int8", batches, prompts, args.steps)
-        del dense, weights
+        other = like(pkg, torch, c, prompts, vocab)
+        for mine, its in zip((decode, prefill), measure(*other)):
+            for k in mine:
+                mine[k][like_name] = its[k]
+        del other
         torch.cuda.empty_cache()
-        rec = {"config": dict(c, vocab=vocab, head_dim=128), "decode": {}, "prefill": {}}
-        for B in batches:
-            byt, dbyt = tovelix_step_bytes(c, B, PROMPT), step_weight_bytes(dc) + B * PROMPT * kv_bytes_per_token(dc)
-            rec["decode"][f"batch{B}"] = {
-                "ms": round(t["decode"][B], 4), "tok_s": round(B * 1e3 / t["decode"][B], 1), "hbm_frac": round(byt / t["decode"][B] / 1e6 / hbm, 4),
-                "dense_w4a16": {"ms": round(u["decode"][B], 4), "tok_s": round(B * 1e3 / u["decode"][B], 1),
-                                "hbm_frac": round(dbyt / u["decode"][B] / 1e6 / hbm, 4)}}
-        for S in prompts:
-            fl = tovelix_prefill_flops(c, S)
-            dfl = 2.0 * S * sum(a * b for a, b in linear_shapes(dc).values()) * n + 2.0 * vocab * c["width"] + n * 2.0 * c["heads"] * 128 * S * (S + 1)
-            rec["prefill"][f"{S}"] = {
-                "ms": round(t["prefill"][S], 3), "tok_s": round(S * 1e3 / t["prefill"][S], 1), "bf16_frac": round(fl / t["prefill"][S] / 1e9 / tf, 4),
-                "dense_w4a16": {"ms": round(u["prefill"][S], 3), "tok_s": round(S * 1e3 / u["prefill"][S], 1),
-                                "bf16_frac": round(dfl / u["prefill"][S] / 1e9 / tf, 4)}}
-        sizes[name] = rec
+        sizes[name] = {"config": dict(c, vocab=vocab), "decode": decode, "prefill": prefill}
     first = next(iter(sizes.values()))["decode"]["batch1"]
-    return {"metric": "Tovelix decode tok/s", "value": first["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": 4,
+    return {"metric": f"{args.model.capitalize()} decode tok/s", "value": first["tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": 4,
             "ms_per_step": first["ms"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-            "config": {"workload": "tovelix", "context": PROMPT, "l2": "the weights of a step exceed the 126 MB L2"},
+            "config": {"workload": args.model, "context": PROMPT, "l2": "the weights of a step exceed the 126 MB L2"},
             "sizes": sizes, "clocks": clocks.summary(), "device_status": pkg.device_status()}
 
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default="dense", choices=["dense", "tovelix"], help="dense: the default workload")
-    ap.add_argument("--size", default="all", choices=["all"] + list(TOVELIX), help="tovelix: one size only")
+    ap.add_argument("--model", default="dense", choices=["dense"] + list(STACKS), help="dense: the default workload")
+    ap.add_argument("--size", default="all", choices=["all"] + list(TOVELIX), help="tovelix, vipelix: one size only")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=8)
@@ -522,9 +602,9 @@ def main():
     cfg = LARGE
     B = args.batch
 
-    if args.model == "tovelix":
+    if args.model in STACKS:
         if rank == 0:
-            print(json.dumps(tovelix_record(args)))
+            print(json.dumps(stack_record(args)))
         return 0
 
     if args.cpu_ops:

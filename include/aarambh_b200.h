@@ -306,11 +306,12 @@ int ab2_moe_forward(const ab2_layer_spec *spec, const ab2_qweight *router, const
  * (kv_rank, normed here with norm_dev), the shared key part (rot_dims) and, with head_gate, heads gate values; ukv is
  * the [heads (dim + vdim), kv_rank] up projection, head by head its key rows and its value rows; tables
  * [positions][rot_dims / 2]; out_dev [nrows * S][heads vdim].  proj_dev may be rewritten.  workspace_dev holds
- * ab2_latent_workspace bytes for nrows * S tokens and `positions` cached ones. */
+ * ab2_latent_workspace bytes for nrows * S tokens and `positions` cached ones; with reuse it still has what an earlier call
+ * derived from the same ukv. */
 int ab2_latent_workspace(const ab2_layer_spec *spec, int tokens, int positions, ab2_dtype dtype, size_t *bytes);
 int ab2_latent_attention(ab2_kv *kv, int layer, const ab2_layer_spec *spec, void *proj_dev, long long stride, const float *norm_dev,
                          const ab2_qweight *ukv, const float *cos_dev, const float *sin_dev, float eps, void *out_dev,
-                         void *workspace_dev, size_t workspace_bytes, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
+                         void *workspace_dev, size_t workspace_bytes, int reuse, int S, int row0, int nrows, ab2_dtype dtype, ab2_stream stream);
 /* out_dev [rows][n] = a N(z) + b N(z^2) + c N(z^3) + e with coef_host = {a, b, c, e} (AB2_FFN_POLY). */
 int ab2_poly_norm(const void *z_dev, void *out_dev, int rows, int n, const float *coef_host, float eps, ab2_dtype dtype, ab2_stream stream);
 

@@ -307,7 +307,7 @@ def bench_stack(pkg, args):
     """The kernels of layer stacks, each in a graph over operands that exceed L2 (several weights or caches
     in turn): dense bf16 linears, mixture of experts, window attention, lightning attention."""
     stream = torch.cuda.Stream()
-    only = args.only.split(",") if args.only else ["linear", "moe", "window", "lightning"]
+    only = args.only.split(",") if args.only else ["linear", "moe", "window", "lightning", "latent"]
 
     def lin(n, k):
         return pkg.QuantLinear.from_bf16(torch.empty((n, k), dtype=torch.bfloat16, device="cuda").normal_().mul_(k ** -0.5))
@@ -341,6 +341,29 @@ def bench_stack(pkg, args):
                     report("mixture of experts (route, gather, gemm_bf16_tc x 2)", t, flops=2.0 * T * top * 3 * d * ff, width=d, E=E, top=top, ff=ff, T=T)
             del layers
     H, G = 32, 8
+    if "latent" in only:
+        rank, rot, dim, vdim = 512, 64, 128, 128
+        norm, tables = torch.ones(rank, device="cuda"), pkg.dispatch.rotation_tables(16384, rot, 1e4)
+        for h in (16, 32):
+            cfg = pkg.StackConfig(64, 64, [(pkg.LatentMixer(h, dim, rot, vdim, rank, 0.07, 1e4, True), None)], 16384)
+            ukv, width = lin(h * (dim + vdim), rank), -(-(h * (dim + rot + 1) + rank + rot) // 8) * 8
+            work = torch.empty(1 << 29, dtype=torch.uint8, device="cuda")
+            for ctx, B in ((512, 1), (512, 32), (4096, 1), (4096, 8), (4096, 32), (16384, 32)):
+                caches = [pkg.KVCache.for_stack(cfg, ctx, B, 512, "bf16") for _ in range(max(1, min(40, math.ceil(400e6 / (B * ctx * 2 * (rank + rot))))))]
+                for c in caches:
+                    c.commit(ctx - 8, 0, B)
+                proj = x_of(B, 1, width)
+                pkg.dispatch.latent_attention(caches[0], cfg, 0, proj, norm, ukv, tables, 1e-5, workspace=work)
+                t = time_graph(lambda: [pkg.dispatch.latent_attention(c, cfg, 0, proj, norm, ukv, tables, 1e-5, workspace=work, reuse=True) for c in caches],
+                               5, stream) / len(caches)
+                report("latent attention, decode (all launches)", t, byt=B * ctx * 2 * (rank + rot) + 2 * h * (dim + vdim) * rank, heads=h, ctx=ctx, B=B)
+                del caches
+            for S in (512, 2048, 8192):
+                cache, proj = pkg.KVCache.for_stack(cfg, S, 1, S, "bf16"), x_of(1, S, width)
+                t = time_graph(lambda: pkg.dispatch.latent_attention(cache, cfg, 0, proj, norm, ukv, tables, 1e-5, workspace=work, reuse=True), 5, stream)
+                report("latent attention, prompt (preparation, projection, attention)", t, flops=h * (dim + rot + vdim) * S * (S + 1.0) + 2.0 * S * h * (dim + vdim) * rank,
+                       heads=h, S=S)
+                del cache
     if "window" in only:
         for W, ctx, B in ((1024, 4096, 1), (1024, 4096, 32), (4096, 8192, 1), (4096, 8192, 32), (0, 32768, 8)):
             cfg = pkg.StackConfig(64, 64, [(pkg.AttentionMixer(H, G, 128, 128, 0.09, W), None)], ctx)
@@ -381,11 +404,14 @@ def bench_stack(pkg, args):
 
 def run_stack_step(pkg, args):
     """Three graph-replayed decode steps (context 512, --batch sequences) or two prefills of --prompt tokens of
-    a Tovelix stack of bench.py's size --size with the layers --pattern: the workload of the stack's profiles."""
+    a stack of bench.py's size --size: Tovelix with the layers --pattern, or (pattern V) two layers of Vipelix.
+    The workload of the stacks' profiles."""
     import bench
-    c = dict(bench.TOVELIX[args.size], layers=args.pattern)
     B, S = (1, args.prompt) if args.prompt else (args.batch, 512)
-    model = bench.build_tovelix(pkg, torch, c, max(S, 32), S + 64)
+    if args.pattern == "V":
+        model = bench.build_vipelix(pkg, torch, dict(bench.VIPELIX[args.size], layers=2, loop=(1, 2, 2)), max(S, 32), S + 64)
+    else:
+        model = bench.build_tovelix(pkg, torch, dict(bench.TOVELIX[args.size], layers=args.pattern), max(S, 32), S + 64)
     cache = model.empty_kv_cache_with_capacity(S + 40, batch=B)
     prompt = torch.randint(0, 32000, (B, S), generator=torch.Generator().manual_seed(1))
     stream = torch.cuda.Stream()
@@ -405,10 +431,10 @@ def run_stack_step(pkg, args):
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("what", choices=["gemv", "gemm", "attention", "prefill_attention", "step", "stack", "stack_step"])
-    ap.add_argument("--size", default="w2048", help="stack_step: a size of bench.py's Tovelix table")
-    ap.add_argument("--pattern", default="LA", help="stack_step: layers, L lightning, A attention")
+    ap.add_argument("--size", default="w2048", help="stack_step: a size of bench.py's tables")
+    ap.add_argument("--pattern", default="LA", help="stack_step: layers, L lightning, A attention; V: two layers of Vipelix")
     ap.add_argument("--prompt", type=int, default=0, help="stack_step: prefill this many tokens (0: decode steps)")
-    ap.add_argument("--only", default=None, help="stack: linear, moe, window, lightning")
+    ap.add_argument("--only", default=None, help="stack: linear, moe, window, lightning, latent")
     ap.add_argument("--layers", type=int, default=2)
     ap.add_argument("--ctx", type=int, default=512)
     ap.add_argument("--batch", type=int, default=1, help="step: sequences decoded together")
