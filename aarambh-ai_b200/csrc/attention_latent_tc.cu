@@ -62,25 +62,6 @@ struct LtSlot {
     }
 };
 
-// M- or N-major operand, 128-byte swizzle: 64 elements of M per row of K, 8 rows a group of 1024 bytes,
-// the next 64 elements `lbo` bytes further.
-__device__ __forceinline__ uint64_t umma_desc_mn(uint32_t saddr, uint32_t lbo) {
-    uint64_t d = 0;
-    d |= (uint64_t)((saddr >> 4) & 0x3FFF);
-    d |= (uint64_t)(lbo >> 4) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
-// One lane of a converged warp, always the same one.
-__device__ __forceinline__ bool elect_one() {
-    uint32_t p;
-    asm volatile("{\n .reg .pred e;\n elect.sync _|e, 0xffffffff;\n selp.u32 %0, 1, 0, e;\n}\n" : "=r"(p));
-    return p;
-}
-// A wait of a whole warp, with one answer for it.
-__device__ __forceinline__ bool warp_wait(uint64_t *bar, uint32_t parity, volatile int *failed) { return __all_sync(0xffffffffu, bar_wait(bar, parity, failed)); }
 constexpr uint32_t LT_IDESC = (1u << 4) | (1u << 7) | (1u << 10);  // f32 sums of bf16 products
 // Barrier of the softmax warps; returns whether any of them passed true.
 __device__ __forceinline__ bool softmax_any(bool p) {

@@ -814,6 +814,7 @@ bool prompt_attention_serves(int dim, int tail, int vdim) {
 }
 
 int prompt_attention(const PromptAttnArgs &a, cudaStream_t s) {
+    if (prompt_tc_serves(a)) return prompt_tc_attention(a, s);
     const int d = a.dim + a.tail_dims;
     cudaError_t e;
     if (d <= 64) e = a.vdim <= 64 ? launch_mma<64, 64>(a, a.heads, 1, s) : launch_mma<64, 128>(a, a.heads, 1, s);

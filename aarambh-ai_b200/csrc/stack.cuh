@@ -87,7 +87,7 @@ static inline size_t latent_part_ml_bytes() { return (size_t)LATENT_PART_TILES *
 
 // Causal attention of a prompt portion's S queries of one sequence over keys and values laid out
 // position by position; the last `tail_dims` dimensions of a key are shared by the heads
-// (attention_window.cu, bf16 only).
+// (bf16 only: on tcgen05 where the shape allows it, else window_attn_mma_kernel).
 struct PromptAttnArgs {
     const __nv_bfloat16 *q, *k, *tail, *v, *gate;   // gate: [S][gate_stride] per head, or null
     long long q_stride, k_stride, tail_stride, v_stride, gate_stride, out_stride;  // between positions
@@ -97,6 +97,8 @@ struct PromptAttnArgs {
     float scale;
 };
 bool prompt_attention_serves(int dim, int tail, int vdim);
+bool prompt_tc_serves(const PromptAttnArgs &a);   // attention_prompt_tc.cu
+int prompt_tc_attention(const PromptAttnArgs &a, cudaStream_t s);
 int prompt_attention(const PromptAttnArgs &a, cudaStream_t s);
 
 // ---- normalisation around the f32 residual stream (ops.cu) -------------------------

@@ -1,6 +1,6 @@
 // tcgen05 / TMA building blocks shared by the W4A16 tensor-memory kernels
 // (internal header): mbarrier helpers with bounded waits, bulk and tensor-map
-// copies, the K-major 128-byte-swizzle shared-memory descriptor, the bf16 MMA
+// copies, the K-major 128-byte-swizzle shared-memory descriptors, the bf16 MMA
 // issue and commit, and the host-side tensor map of a [rows][K] bf16 matrix.
 #pragma once
 
@@ -90,6 +90,26 @@ __device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t adesc, uint6
 __device__ __forceinline__ void umma_commit(uint64_t *bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n" ::"r"(sptr(bar)) : "memory");
 }
+
+// M- or N-major operand, 128-byte swizzle: 64 elements of M per row of K, 8 rows a group of 1024 bytes,
+// the next 64 elements `lbo` bytes further.
+__device__ __forceinline__ uint64_t umma_desc_mn(uint32_t saddr, uint32_t lbo) {
+    uint64_t d = 0;
+    d |= (uint64_t)((saddr >> 4) & 0x3FFF);
+    d |= (uint64_t)(lbo >> 4) << 16;
+    d |= (uint64_t)(1024 >> 4) << 32;
+    d |= (uint64_t)1 << 46;
+    d |= (uint64_t)2 << 61;
+    return d;
+}
+// One lane of a converged warp, always the same one.
+__device__ __forceinline__ bool elect_one() {
+    uint32_t p;
+    asm volatile("{\n .reg .pred e;\n elect.sync _|e, 0xffffffff;\n selp.u32 %0, 1, 0, e;\n}\n" : "=r"(p));
+    return p;
+}
+// A wait of a whole warp, with one answer for it.
+__device__ __forceinline__ bool warp_wait(uint64_t *bar, uint32_t parity, volatile int *failed) { return __all_sync(0xffffffffu, bar_wait(bar, parity, failed)); }
 
 __device__ __forceinline__ uint32_t bf16x2_add_(uint32_t a, uint32_t b) {
     uint32_t d;
