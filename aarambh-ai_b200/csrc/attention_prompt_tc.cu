@@ -50,12 +50,16 @@ struct PtArgs {
     c(v[16]), c(v[17]), c(v[18]), c(v[19]), c(v[20]), c(v[21]), c(v[22]), c(v[23]), c(v[24]), c(v[25]), c(v[26]), c(v[27]), c(v[28]), c(v[29]), c(v[30]), c(v[31])
 // 32 columns of the warp's lanes; the registers pass through the wait, so that nothing computed from them can move
 // ahead of it.
-__device__ __forceinline__ void tmem_ld32(uint32_t (&v)[32], uint32_t addr) {
+__device__ __forceinline__ void tmem_ld32_start(uint32_t (&v)[32], uint32_t addr) {
     asm volatile(
         "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
         "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n"
         : PT_REGS32("=r", v) : "r"(addr));
-    asm volatile("tcgen05.wait::ld.sync.aligned;\n" : PT_REGS32("+r", v)::"memory");
+}
+__device__ __forceinline__ void tmem_ld32_wait(uint32_t (&v)[32]) { asm volatile("tcgen05.wait::ld.sync.aligned;\n" : PT_REGS32("+r", v)::"memory"); }
+__device__ __forceinline__ void tmem_ld32(uint32_t (&v)[32], uint32_t addr) {
+    tmem_ld32_start(v, addr);
+    tmem_ld32_wait(v);
 }
 __device__ __forceinline__ void tmem_st32(uint32_t addr, const uint32_t (&v)[32]) {
     asm volatile(
@@ -74,6 +78,60 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, u
         "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
         " tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n" ::
             "r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
+}
+
+// One tile of keys for the warp's 32 queries, a lane each: scores to weights in tensor memory.  With EDGE the keys
+// past `lim` are out of sight.  o_blocks blocks of 32 columns hold sums so far.
+template <bool EDGE>
+__device__ __forceinline__ void softmax_tile(uint32_t s_addr, uint32_t o_addr, float sl, int lim, int o_blocks, float &top, float &sum) {
+    // two buffers: the next 32 scores are on their way while these are looked at
+    uint32_t v[2][32];
+    float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+    tmem_ld32_start(v[0], s_addr);
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+        tmem_ld32_wait(v[c & 1]);
+        tmem_ld32_start(v[(c + 1) & 1], s_addr + 32 * ((c + 1) & 3));  // the last one fetches the first again
+#pragma unroll
+        for (int k = 0; k < 32; ++k) mx[k & 3] = fmaxf(mx[k & 3], EDGE && 32 * c + k > lim ? -INFINITY : __uint_as_float(v[c & 1][k]));
+    }
+    tmem_ld32_wait(v[0]);
+    const float best = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * sl;  // the scale is positive
+    const float now = best > top + PT_SLACK ? best : top;
+    if (__any_sync(0xffffffffu, now != top)) {
+        const float corr = ex2(top - now);
+        sum *= corr;
+        top = now;
+        // the scores came after the products of this half's last tile: its sums stand still
+#pragma unroll 1
+        for (int c = 0; c < o_blocks; ++c) {
+            uint32_t o[32];
+            tmem_ld32(o, o_addr + 32 * c);
+#pragma unroll
+            for (int k = 0; k < 32; ++k) o[k] = __float_as_uint(__uint_as_float(o[k]) * corr);
+            tmem_st32(o_addr + 32 * c, o);
+        }
+    }
+    float part_sum[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+        if (c > 0) tmem_ld32_wait(v[c & 1]);
+        if (c < 3) tmem_ld32_start(v[(c + 1) & 1], s_addr + 32 * (c + 1));
+        uint32_t w[32];
+#pragma unroll
+        for (int k = 0; k < 32; k += 2) {
+            float x = ex2(fmaf(__uint_as_float(v[c & 1][k]), sl, -top)), y = ex2(fmaf(__uint_as_float(v[c & 1][k + 1]), sl, -top));
+            if (EDGE && 32 * c + k > lim) x = 0.f;
+            if (EDGE && 32 * c + k + 1 > lim) y = 0.f;
+            part_sum[(k >> 1) & 3] += x + y;
+            const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+            w[k >> 1] = *reinterpret_cast<const uint32_t *>(&h);
+            const __nv_bfloat162 l = __floats2bfloat162_rn(x - __uint_as_float(w[k >> 1] << 16), y - __uint_as_float(w[k >> 1] & 0xffff0000u));
+            w[16 + (k >> 1)] = *reinterpret_cast<const uint32_t *>(&l);
+        }
+        tmem_st32(s_addr + 32 * c, w);
+    }
+    sum += (part_sum[0] + part_sum[1]) + (part_sum[2] + part_sum[3]);
 }
 
 __global__ void __launch_bounds__(PT_THREADS, 1)
@@ -133,7 +191,6 @@ prompt_tc_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
     const uint32_t tmem = sh->tmem_base, tmem_o = tmem + 2 * PT_KEYS;  // O_0 and O_1 128 columns apart
     constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 4) << 24);
-
     if (warp == 0) {
         // ---------------------------------------------------------- TMA producer
         if (lane == 0)
@@ -191,61 +248,14 @@ prompt_tc_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
         const float sl = a.scale * 1.44269504088896341f;  // scores in powers of two
         float top = -1e30f, sum = 0.f;
         bool ok = true;
-        uint32_t v[32];
         for (int j = part; j < tiles; j += 2) {
             ok = warp_wait(&sh->sfull[part], (j >> 1) & 1, failed);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const bool edge = (j + 1) * PT_KEYS - 1 > a.first + q_lo;
             const int lim = pos - j * PT_KEYS;  // the last key of the tile in sight
-            float mx = -INFINITY;
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                tmem_ld32(v, s_addr + 32 * c);
-                if (edge) {
-#pragma unroll
-                    for (int k = 0; k < 32; ++k) mx = fmaxf(mx, 32 * c + k <= lim ? __uint_as_float(v[k]) : -INFINITY);
-                } else {
-#pragma unroll
-                    for (int k = 0; k < 32; ++k) mx = fmaxf(mx, __uint_as_float(v[k]));
-                }
-            }
-            const float now = mx * sl > top + PT_SLACK ? mx * sl : top;  // the scale is not negative
-            if (__any_sync(0xffffffffu, now != top)) {
-                const float corr = ex2(top - now);
-                sum *= corr;
-                top = now;
-                if (j >= 2) {  // the scores came after the products of this half's last tile: its sums stand still
-#pragma unroll 1
-                    for (int c = 0; c < p.v_boxes * 2; ++c) {
-                        tmem_ld32(v, o_addr + 32 * c);
-#pragma unroll
-                        for (int k = 0; k < 32; ++k) v[k] = __float_as_uint(__uint_as_float(v[k]) * corr);
-                        tmem_st32(o_addr + 32 * c, v);
-                    }
-                }
-            }
-            float part_sum[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                tmem_ld32(v, s_addr + 32 * c);
-                uint32_t w[32];
-#pragma unroll
-                for (int k = 0; k < 32; k += 2) {
-                    float x = ex2(fmaf(__uint_as_float(v[k]), sl, -top)), y = ex2(fmaf(__uint_as_float(v[k + 1]), sl, -top));
-                    if (edge) {
-                        if (32 * c + k > lim) x = 0.f;
-                        if (32 * c + k + 1 > lim) y = 0.f;
-                    }
-                    part_sum[(k >> 1) & 3] += x + y;
-                    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-                    w[k >> 1] = *reinterpret_cast<const uint32_t *>(&h);
-                    const __nv_bfloat162 l = __floats2bfloat162_rn(x - __uint_as_float(w[k >> 1] << 16), y - __uint_as_float(w[k >> 1] & 0xffff0000u));
-                    w[16 + (k >> 1)] = *reinterpret_cast<const uint32_t *>(&l);
-                }
-                tmem_st32(s_addr + 32 * c, w);
-            }
-            sum += (part_sum[0] + part_sum[1]) + (part_sum[2] + part_sum[3]);
+            if (edge) softmax_tile<true>(s_addr, o_addr, sl, lim, j >= 2 ? p.v_boxes * 2 : 0, top, sum);
+            else softmax_tile<false>(s_addr, o_addr, sl, lim, j >= 2 ? p.v_boxes * 2 : 0, top, sum);
             asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
             __syncwarp();
@@ -270,7 +280,7 @@ prompt_tc_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant
             __nv_bfloat16 *dst = a.out + (size_t)qi * a.out_stride + (size_t)head * a.vdim;
 #pragma unroll 1
             for (int c = part; c < p.v_boxes * 2; c += 2) {
-                uint32_t w[32];
+                uint32_t v[32], w[32];
                 __syncwarp();
                 tmem_ld32(v, tmem_o + quad_addr + 32 * c);
                 if (tiles > 1) tmem_ld32(w, tmem_o + quad_addr + 128 + 32 * c);
