@@ -379,9 +379,9 @@ __global__ void poly_norm_kernel(PolyNormArgs p) {
     const T *z = (const T *)p.z + (size_t)blockIdx.x * p.n;
     T *out = (T *)p.out + (size_t)blockIdx.x * p.n;
     struct alignas(V * sizeof(T)) Vec { T e[V]; };
+    constexpr int KEEP = 4;  // vectors of a thread that stay in registers
     float s2 = 0.f, s4 = 0.f, s6 = 0.f;
-    for (int i = threadIdx.x; i < p.n / V; i += blockDim.x) {
-        const Vec q = reinterpret_cast<const Vec *>(z)[i];
+    auto take = [&](const Vec &q) {
 #pragma unroll
         for (int j = 0; j < V; ++j) {
             const float v = to_f32(q.e[j]), w = v * v;
@@ -389,7 +389,16 @@ __global__ void poly_norm_kernel(PolyNormArgs p) {
             s4 = fmaf(w, w, s4);
             s6 = fmaf(w * w, w, s6);
         }
-    }
+    };
+    const int nv = p.n / V;
+    Vec keep[KEEP];
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+        if (threadIdx.x + k * blockDim.x < nv) keep[k] = reinterpret_cast<const Vec *>(z)[threadIdx.x + k * blockDim.x];
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+        if (threadIdx.x + k * blockDim.x < nv) take(keep[k]);
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < nv; i += blockDim.x) take(reinterpret_cast<const Vec *>(z)[i]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
         s2 += __shfl_xor_sync(0xffffffffu, s2, o);
@@ -403,8 +412,7 @@ __global__ void poly_norm_kernel(PolyNormArgs p) {
     for (int i = 0; i < (int)(blockDim.x >> 5); ++i) { s2 += sums[0][i]; s4 += sums[1][i]; s6 += sums[2][i]; }
     const float n = (float)p.n;
     const float a = p.a / sqrtf(s2 / n + p.eps), b = p.b / sqrtf(s4 / n + p.eps), c = p.c / sqrtf(s6 / n + p.eps);
-    for (int i = threadIdx.x; i < p.n / V; i += blockDim.x) {
-        const Vec q = reinterpret_cast<const Vec *>(z)[i];
+    auto give = [&](const Vec &q, int i) {
         Vec r;
 #pragma unroll
         for (int j = 0; j < V; ++j) {
@@ -412,12 +420,16 @@ __global__ void poly_norm_kernel(PolyNormArgs p) {
             r.e[j] = from_f32<T>(fmaf(v, fmaf(v, fmaf(v, c, b), a), p.e));
         }
         reinterpret_cast<Vec *>(out)[i] = r;
-    }
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+        if (threadIdx.x + k * blockDim.x < nv) give(keep[k], threadIdx.x + k * blockDim.x);
+    for (int i = threadIdx.x + KEEP * blockDim.x; i < nv; i += blockDim.x) give(reinterpret_cast<const Vec *>(z)[i], i);
 }
 
 int launch_poly_norm(const PolyNormArgs &p, int rows, ab2_dtype dtype, cudaStream_t s) {
     const bool vec = p.n % 8 == 0;
-    const int threads = std::min(1024, std::max(128, (p.n / 16 + 31) / 32 * 32));
+    const int threads = std::min(1024, std::max(128, (p.n / (vec ? 32 : 16) + 31) / 32 * 32));
     cudaError_t e;
     if (dtype == AB2_F32) e = vec ? launch_kernel(poly_norm_kernel<float, 4>, dim3(rows), dim3(threads), 0, s, p) : launch_kernel(poly_norm_kernel<float, 1>, dim3(rows), dim3(threads), 0, s, p);
     else e = vec ? launch_kernel(poly_norm_kernel<__nv_bfloat16, 8>, dim3(rows), dim3(threads), 0, s, p) : launch_kernel(poly_norm_kernel<__nv_bfloat16, 1>, dim3(rows), dim3(threads), 0, s, p);

@@ -109,6 +109,20 @@ def test_a_late_key_towers_over_the_others(H, dim, rot, vdim, rank):
         assert rel_err(got[S - 2, h], x.want[S - 2, h]) < 3e-2, h
 
 
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,first", [(8, 128, 64, 128, 128, 0), (7, 40, 24, 72, 64, 0), (8, 64, 0, 64, 96, 133), (6, 136, 40, 64, 64, 5)])
+def test_long_prompt_portions(H, dim, rot, vdim, rank, first):
+    """Many key tiles per query, the highest scores in early, middle and late ones, at the tiles' edges."""
+    T = 900
+    at = T - 2
+    x = LatentCase(H, dim, rot, vdim, rank, T, at, (0, 127, 128, 511, 640, 767, 895, at - 1)[:H], 21, first=T - 150)
+    for cuts in ([(0, T)], [(0, first), (first, T)], [(0, 300), (300, 429), (429, T)]):
+        cuts = [c for c in cuts if c[1] > c[0]]
+        got = x.run(x.cache(torch.bfloat16), cuts, torch.bfloat16)[T - 150:]
+        assert rel_err(got, x.want) < 1.5e-2, cuts
+        for h in range(H):
+            assert rel_err(got[at - T + 150, h], x.want[at - T + 150, h]) < 3e-2, (cuts, h)
+
+
 @pytest.mark.parametrize("first", [0, 37])
 def test_prompt_projected_some_heads_at_a_time(first):
     """A workspace that holds the keys and values of three heads only, and one that holds none."""
