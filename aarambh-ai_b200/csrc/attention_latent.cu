@@ -43,13 +43,24 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a, T *qx) {
         const float v = to_f32(c[i]);
         sum = fmaf(v, v, sum);
     }
-    for (int i = threadIdx.x; i < (a.H + 1) * half; i += 256) {
-        const int h = i / half, j = i % half;
-        const T *src = h < a.H ? q + (size_t)h * (a.dim + a.rot) + a.dim : kr;
-        T *out = h == a.H ? dst + a.rank : qx ? qx + (tok * a.H + h) * l.kds + a.rank : q + (size_t)h * (a.dim + a.rot) + a.dim;
-        const float u = to_f32(src[2 * j]), v = to_f32(src[2 * j + 1]), cs = ct[j], sn = st[j];
-        out[2 * j] = from_f32<T>(u * cs - v * sn);
-        out[2 * j + 1] = from_f32<T>(v * cs + u * sn);
+    // a warp takes every eighth head (the key part counts as the last); a lane keeps its angles for all of them
+    struct alignas(2 * sizeof(T)) Pair { T u, v; };
+    const bool paired = ((a.dim | (int)a.stride | a.rank) & 1) == 0;  // pairs lie on their own size (rot and kds are even)
+    for (int j = threadIdx.x & 31; j < half; j += 32) {
+        const float cs = ct[j], sn = st[j];
+#pragma unroll 4
+        for (int h = threadIdx.x >> 5; h <= a.H; h += 8) {
+            const T *src = (h < a.H ? q + (size_t)h * (a.dim + a.rot) + a.dim : kr) + 2 * j;
+            T *out = (h == a.H ? dst + a.rank : qx ? qx + (tok * a.H + h) * l.kds + a.rank : q + (size_t)h * (a.dim + a.rot) + a.dim) + 2 * j;
+            Pair p;
+            if (paired) p = *reinterpret_cast<const Pair *>(src);
+            else { p.u = src[0]; p.v = src[1]; }
+            const float u = to_f32(p.u), v = to_f32(p.v);
+            p.u = from_f32<T>(u * cs - v * sn);
+            p.v = from_f32<T>(v * cs + u * sn);
+            if (paired) *reinterpret_cast<Pair *>(out) = p;
+            else { out[0] = p.u; out[1] = p.v; }
+        }
     }
     const int used = a.rank + a.rot, pad = l.kds - used;
     if (qx)
