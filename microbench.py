@@ -347,7 +347,7 @@ def bench_stack(pkg, args):
         for h in (16, 32):
             cfg = pkg.StackConfig(64, 64, [(pkg.LatentMixer(h, dim, rot, vdim, rank, 0.07, 1e4, True), None)], 16384)
             ukv, width = lin(h * (dim + vdim), rank), -(-(h * (dim + rot + 1) + rank + rot) // 8) * 8
-            work = torch.empty(1 << 29, dtype=torch.uint8, device="cuda")
+            work = torch.empty(1 << 30, dtype=torch.uint8, device="cuda")
             for ctx, B in ((512, 1), (512, 32), (4096, 1), (4096, 8), (4096, 32), (16384, 32)):
                 caches = [pkg.KVCache.for_stack(cfg, ctx, B, 512, "bf16") for _ in range(max(1, min(40, math.ceil(400e6 / (B * ctx * 2 * (rank + rot))))))]
                 for c in caches:

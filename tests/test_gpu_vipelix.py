@@ -60,7 +60,7 @@ class LatentCase:
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,dim,rot,vdim,rank,T", [(4, 32, 16, 48, 96, 200), (3, 16, 8, 24, 40, 150), (40, 24, 8, 16, 64, 140), (1, 128, 64, 128, 512, 150),
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,T", [(4, 40, 16, 56, 104, 200), (3, 16, 8, 24, 40, 150), (40, 24, 8, 16, 64, 140), (1, 128, 64, 128, 512, 150),
                                                    (5, 20, 6, 18, 44, 90), (2, 7, 2, 5, 9, 70), (2, 40, 0, 32, 128, 140), (33, 8, 8, 8, 72, 135),
                                                    (2, 64, 32, 64, 640, 70), (6, 144, 40, 72, 320, 133)])
 def test_latent_attention(dtype, H, dim, rot, vdim, rank, T):
